@@ -44,7 +44,8 @@ enum {
   PIEH_EPI_GLU = 4,      /* gated pair (pieh_linear_glu only): out [M, N / 2]                                        */
   PIEH_EPI_SIGMUL = 5,   /* y <- y * sigmoid(gate[m, n])   (pieh_linear_batched only)                                */
   PIEH_EPI_TANH = 6,     /* y <- tanh(y)                   (pieh_linear_act only)                                    */
-  PIEH_EPI_XIELU = 7     /* y <- a y^2 + y / 2 (y > 0),  b (e^y - 1 - y) + y / 2 (y <= 0)   (pieh_linear_act only)    */
+  PIEH_EPI_XIELU = 7,    /* y <- a y^2 + y / 2 (y > 0),  b (e^y - 1 - y) + y / 2 (y <= 0)   (pieh_linear_act only)    */
+  PIEH_EPI_GELU = 8      /* y <- y / 2 (1 + tanh(sqrt(2 / pi) (y + 0.044715 y^3)))          (pieh_linear_act only)    */
 };
 
 /* ragged step descriptor, shared by the recurrent and the attention operators (all arrays int32, device) */
@@ -71,7 +72,7 @@ int pieh_linear(void* out, int out_dtype, long long out_ld, const void* x, int x
                 int w_dtype, const float* bias, int M, int N, int K, int epilogue, float epi_a, const float* mix,
                 const float* outw, int S, void* stream);
 
-/* pieh_linear with an activation that takes up to two constants: NONE, RELU2, TANH, or XIELU with a = act_a, b = act_b
+/* pieh_linear with an activation that takes up to two constants: NONE, RELU2, TANH, GELU, or XIELU with a = act_a, b = act_b
  * (the caller passes the finished coefficients, e.g. softplus of learned numbers). */
 int pieh_linear_act(void* out, int out_dtype, long long out_ld, const void* x, int x_dtype, long long x_ld, const void* w,
                     int w_dtype, const float* bias, int M, int N, int K, int act, float act_a, float act_b, void* stream);
@@ -205,6 +206,9 @@ typedef struct pieh_bias_attn {
   int sigmoid;             /* 1: no softmax -- a visible key weighs sigmoid(s_ij + score_bias[h]), the weights are not normalised
                               over the keys and there is no sink */
   const float* score_bias; /* [H] added to the score inside the sigmoid (NULL: none) */
+  long long q_ld;          /* floats between two tokens' queries in pieh_bias_attn_run (0: H d) */
+  long long v_ld;          /* elements between two positions' value rows (0: G dv).  With G = 1 and v_pages == k_pages, v_ld = d:
+                              the values are the leading dv features of the cached key rows (latent attention) */
 } pieh_bias_attn;
 /* q_out fp32 [T, H, d]; k' and v appended to the pages at each row's position.  Rotation (after the norms) turns the pair
  * (u, v) = (x[i], x[i + rot_dims / 2]) into (u cos - v sin, v cos + u sin). */
@@ -236,6 +240,13 @@ typedef struct pieh_moe_plan {
   int32_t* counters;     /* [2 * E + 2] scratch */
   int softmax_top;       /* 1: no groups, no sigmoid: the `top` largest LOGITS are chosen and weigh softmax over the chosen
                             logits only (times scale) */
+  /* optional pieces (all zero / NULL: off) of the grouped choice */
+  int softmax_all;       /* 1: s = softmax over ALL E + identity logits instead of the sigmoid */
+  const float* correction; /* [E + identity] added to s for choosing (group scores included); the weights use s without it */
+  int group_best;        /* 1: a group scores its single best choice score instead of the sum of its two best */
+  int identity;          /* the last `identity` router outputs (numbers E .. E + identity - 1; z and the groups span all of them)
+                            are identity experts without matrices: such a pair takes no slot, pair_slot = -1 (pieh_sum_norm
+                            understands it); slots past the last real one have slot_expert = -1 */
 } pieh_moe_plan;
 int pieh_moe_route(const float* z, long long ld, const pieh_moe_plan* p, int T, void* stream);
 /* Grouped product over the slots: out[s, :] = x[row(s), :] W_e(s)^T with W_e = w + e * w_stride elements, row(s) =
@@ -294,6 +305,66 @@ int pieh_latent_prepare(void* cq_out, int out_dtype, const float* proj, long lon
 int pieh_sandwich_add(float* x, const float* y, const pieh_mix_sum* mix, const float* post_w, float mult,
                       const float* add_rows, const float* add_vec, void* h, int h_dtype, const float* next_w, float eps,
                       int T, int W, void* stream);
+
+/* ---- post-norm residual whose norm REPLACES it, and the pair embedding --------------------------------------------------------
+ *   s = alpha * x[t, :] + (y ? y[t, :] : mixture),   x[t, :] = s / sqrt(mean(s^2) + eps) * norm_w,   act[t, :] = x[t, :]
+ * The mixture is that of pieh_postnorm_add (a NULL shared_gate: the shared rows count fully), except that part_row < 0 stands
+ * for x[t, :] itself (an identity expert).  x fp32 [T, W]; act in the act dtype, may be NULL. */
+int pieh_sum_norm(float* x, void* act, int act_dtype, const float* y, const pieh_mix_sum* mix, const float* norm_w,
+                  float alpha, float eps, int T, int W, void* stream);
+/* x[t, :] = table[token] * scale + pairs[row],  row = (previous token * mul_prev + token * mul_cur) mod buckets, or the extra
+ * row `buckets` for a sequence's first token.  pairs [buckets + 1, W] in the table's dtype, or NULL (then nothing is added and
+ * prev is not touched).  prev int32 [slots]: the last token of every sequence, read for the first row of a portion and moved
+ * on.  act (may be NULL): x in the act dtype. */
+int pieh_embed_pairs(float* x, void* act, int act_dtype, const void* table, const void* pairs, int table_dtype,
+                     const int32_t* tokens, float scale, long long mul_prev, long long mul_cur, int buckets, int32_t* prev, int W, int vocab,
+                     const pieh_batch* b, void* stream);
+
+/* ---- gated linear attention: a matrix state with a decay per key channel -------------------------------------------------------
+ * proj fp32 [T, ld] holds q at q_off, k at k_off (H dk each), v at v_off (H dv).
+ *   S_t = diag(a_t) S_(t-1) + k_t v_t^T   (S [dk, dv] per head),   o_t = q_scale * S_t^T q_t */
+typedef struct pieh_gla {
+  int H, dk, dv;           /* dk <= 512 */
+  long long q_off, k_off, v_off;
+  float q_scale;
+  float* state;            /* [slots, H, dk, dv] fp32: read unless the sequence has no context, written back at the end */
+} pieh_gla;
+/* decay[t, c] = sigmoid(bias[c] + sum_r low[t, r] w2t[r, c])^inv_tau, low = proj columns low_off .. low_off + rank - 1;
+ * w2t fp32 [rank, C], C = H dk. */
+int pieh_gla_decay(float* decay, const float* proj, long long ld, long long low_off, int rank, const float* w2t,
+                   const float* bias, float inv_tau, int C, int T, void* stream);
+/* o fp32 [T, H, dv].  scratch NULL: one pass per sequence.  Otherwise portions of more than 64 * seg_tiles rows are cut into
+ * segments of seg_tiles 64-row tiles that are scanned side by side; scratch holds
+ * ((n_tiles - 1) / seg_tiles + n_seq) * H * dk * (dv + 1) floats. */
+int pieh_gla_scan(float* o, const float* proj, long long ld, const float* decay, const pieh_gla* d, const pieh_batch* b,
+                  float* scratch, int seg_tiles, void* stream);
+/* One row per sequence (b->T == b->n_seq): decays, update, read-out, out[t, h, :] = o / sqrt(mean(o^2) + eps) * norm_w *
+ * silu(proj[t, g_off + h dv ...]) in one launch.  norm_w [dv], shared by the heads; dv <= 1024; out act [T, H dv]. */
+int pieh_gla_step(void* out, int out_dtype, const float* proj, long long ld, long long low_off, int rank, const float* w2t,
+                  const float* bias, float inv_tau, long long g_off, const float* norm_w, float eps, const pieh_gla* d,
+                  const pieh_batch* b, void* stream);
+
+/* ---- latent attention with a rotated part beside the latent -----------------------------------------------------------------
+ * proj fp32 [T, ld]: head h's query starts at q_off + h q_head, its positional part (rot_dim features) rot_at further on; the key
+ * / value latent (kv_rank features) is at kv_off and is followed by ONE positional key part (rot_dim) shared by all heads.
+ *   latent -> rms norm with a plain weight -> pages [pages, 64, kv_rank + rot_dim], the rotated key part behind it
+ *   query's positional part, rotated -> q_rot[t * q_rot_ld + h * q_rot_head + f]   (may be its own place in proj)
+ *   query's leading rot_at features  -> q_plain (act [T, H, rot_at]; NULL: skipped)
+ * The leading rot_n features of the positional parts rotate (feature i with i + rot_n / 2, rot_cs as in pieh_bias_attn). */
+typedef struct pieh_latent_rot {
+  int H, kv_rank, rot_dim, rot_n;
+  long long q_off, q_head, rot_at, kv_off;
+  const float* kv_norm;
+  float eps;
+  const float* rot_cs;
+  float* q_rot;
+  long long q_rot_ld, q_rot_head;
+  void* q_plain;
+  int q_plain_dtype;
+  void* pages;
+  int kv_dtype;
+} pieh_latent_rot;
+int pieh_latent_rot_prepare(const float* proj, long long ld, const pieh_latent_rot* a, const pieh_batch* b, void* stream);
 
 /* out[t, c] = norm-and-gate of x[t, :] in `groups` equal parts of group_size features, each by its own root mean square:
  *   gate_first 0:  x / rms(x) * w * f(gate)          gate_first 1:  (x f(gate)) / rms(x f(gate)) * w

@@ -168,7 +168,8 @@ class HybBiasAttn(C.Structure):
                 ("v_pages", C.c_void_p), ("kv_dtype", C.c_int),
                 # optional pieces, zero / NULL = off
                 ("sinks", C.c_void_p), ("gate_heads", C.c_int), ("rot_dims", C.c_int), ("rot_cs", C.c_void_p),
-                ("v_mix", C.c_void_p), ("v_keep", C.c_void_p), ("sigmoid", C.c_int), ("score_bias", C.c_void_p)]
+                ("v_mix", C.c_void_p), ("v_keep", C.c_void_p), ("sigmoid", C.c_int), ("score_bias", C.c_void_p),
+                ("q_ld", C.c_longlong), ("v_ld", C.c_longlong)]
 
 
 class HybMixSum(C.Structure):
@@ -181,7 +182,9 @@ class HybMoePlan(C.Structure):
     """pieh_moe_plan"""
     _fields_ = [("E", C.c_int), ("top", C.c_int), ("n_groups", C.c_int), ("keep_groups", C.c_int), ("scale", C.c_float),
                 ("slot_row", C.c_void_p), ("slot_expert", C.c_void_p), ("pair_slot", C.c_void_p), ("pair_w", C.c_void_p),
-                ("tiles64", C.c_void_p), ("tiles128", C.c_void_p), ("counters", C.c_void_p), ("softmax_top", C.c_int)]
+                ("tiles64", C.c_void_p), ("tiles128", C.c_void_p), ("counters", C.c_void_p), ("softmax_top", C.c_int),
+                # optional pieces, zero / NULL = off
+                ("softmax_all", C.c_int), ("correction", C.c_void_p), ("group_best", C.c_int), ("identity", C.c_int)]
 
 
 class HybCanon(C.Structure):
@@ -204,10 +207,26 @@ class HybSsd(C.Structure):
                 ("A_log", C.c_void_p), ("D", C.c_void_p), ("conv_state", C.c_void_p), ("state", C.c_void_p)]
 
 
+class HybGla(C.Structure):
+    """pieh_gla"""
+    _fields_ = [("H", C.c_int), ("dk", C.c_int), ("dv", C.c_int), ("q_off", C.c_longlong), ("k_off", C.c_longlong),
+                ("v_off", C.c_longlong), ("q_scale", C.c_float), ("state", C.c_void_p)]
+
+
+class HybLatentRot(C.Structure):
+    """pieh_latent_rot"""
+    _fields_ = [("H", C.c_int), ("kv_rank", C.c_int), ("rot_dim", C.c_int), ("rot_n", C.c_int), ("q_off", C.c_longlong),
+                ("q_head", C.c_longlong), ("rot_at", C.c_longlong), ("kv_off", C.c_longlong), ("kv_norm", C.c_void_p),
+                ("eps", C.c_float), ("rot_cs", C.c_void_p), ("q_rot", C.c_void_p), ("q_rot_ld", C.c_longlong),
+                ("q_rot_head", C.c_longlong), ("q_plain", C.c_void_p), ("q_plain_dtype", C.c_int), ("pages", C.c_void_p),
+                ("kv_dtype", C.c_int)]
+
+
 _PB, _PD, _PA = C.POINTER(HybBatch), C.POINTER(HybDelta), C.POINTER(HybAttn)
 _PBA, _PMS, _PMP = C.POINTER(HybBiasAttn), C.POINTER(HybMixSum), C.POINTER(HybMoePlan)
 _PCN = C.POINTER(HybCanon)
 _PGD, _PSS = C.POINTER(HybGdelta), C.POINTER(HybSsd)
+_PGL, _PLR = C.POINTER(HybGla), C.POINTER(HybLatentRot)
 # libpie_b200_hybrid.so: every symbol include/pie_b200_hybrid.h declares (tests check this), + the page allocator
 HYBRID_SIGNATURES = {
     "pieh_abi_version": (_i, []),
@@ -243,11 +262,17 @@ HYBRID_SIGNATURES = {
     "pieh_gdelta_scan": (_i, [_vp, _vp, _ll, _vp, _vp, _vp, _PGD, _PB, _vp]),
     "pieh_ssd_prepare": (_i, [_vp, _vp, _vp, _ll, _PSS, _PB, _vp]),
     "pieh_ssd_scan": (_i, [_vp, _vp, _vp, _PSS, _PB, _vp]),
+    "pieh_sum_norm": (_i, [_vp, _vp, _i, _vp, _PMS, _vp, _f, _f, _i, _i, _vp]),
+    "pieh_embed_pairs": (_i, [_vp, _vp, _i, _vp, _vp, _i, _vp, _f, _ll, _ll, _i, _vp, _i, _i, _PB, _vp]),
+    "pieh_gla_decay": (_i, [_vp, _vp, _ll, _ll, _i, _vp, _vp, _f, _i, _i, _vp]),
+    "pieh_gla_scan": (_i, [_vp, _vp, _ll, _vp, _PGL, _PB, _vp, _i, _vp]),
+    "pieh_gla_step": (_i, [_vp, _i, _vp, _ll, _ll, _i, _vp, _vp, _f, _ll, _vp, _f, _PGL, _PB, _vp]),
+    "pieh_latent_rot_prepare": (_i, [_vp, _ll, _PLR, _PB, _vp]),
     "pieh_moe_route": (_i, [_vp, _ll, _PMP, _i, _vp]),
     "pieh_moe_linear": (_i, [_vp, _i, _ll, _vp, _i, _ll, _vp, _i, _ll, _i, _i, _i, _i, _i, _f, _f, _f, _PMP, _vp]),
 }
 HYBRID_LIB_PATH = os.environ.get("PIE_HYBRID_LIB") or os.path.join(_HERE, "libpie_b200_hybrid.so")
-EPI_NONE, EPI_RELU2, EPI_SOFTCAP, EPI_STREAMS, EPI_GLU, EPI_SIGMUL, EPI_TANH, EPI_XIELU = 0, 1, 2, 3, 4, 5, 6, 7
+EPI_NONE, EPI_RELU2, EPI_SOFTCAP, EPI_STREAMS, EPI_GLU, EPI_SIGMUL, EPI_TANH, EPI_XIELU, EPI_GELU = range(9)
 
 _lib = None
 _hyb = None

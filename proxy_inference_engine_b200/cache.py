@@ -206,7 +206,8 @@ class HybridCache:
       by the page ids of ONE ``paging.PageAllocator`` (a page id names the same 64 positions in every layer's pools);
     * recurrent layers: per state slot the matrix state ``[H, dk, dv]`` and the convolution history ``[taps - 1, C]``, fp32;
     * a spec of the form ``{"pages": {name: shape}, "slots": {name: shape}}`` names its pools and slot tensors itself (a
-      layer may hold both: attention pages beside a convolution history).
+      layer may hold both: attention pages beside a convolution history); ``"int_slots"`` names int32 slot tensors (a
+      sequence's last token, say -- a spec need not belong to a layer).
 
     ``admit`` gives a sequence a slot, ``reserve`` grows its page list to cover a length, ``release`` hands both back
     (LIFO, so the next sequence re-uses them).  Nothing is cleared on re-use: a recurrent operator starts a sequence with
@@ -225,7 +226,7 @@ class HybridCache:
         self.layers = []
         self.slot_keys = {"state", "conv"}     # entries that live in state slots (what a replayed step must put back)
         for spec in layer_specs:
-            if "pages" in spec or "slots" in spec:
+            if "pages" in spec or "slots" in spec or "int_slots" in spec:
                 # the general form: named page pools [pages, 64, *shape] in the act dtype and named per-slot tensors
                 # [slots, *shape] in fp32, whatever mixture of the two a layer needs
                 entry = {}
@@ -233,6 +234,9 @@ class HybridCache:
                     entry[name] = torch.zeros((self.n_pages, self.page_size, *shape), dtype=act_dtype, device=device)
                 for name, shape in (spec.get("slots") or {}).items():
                     entry[name] = torch.zeros((self.max_seqs, *shape), dtype=torch.float32, device=device)
+                    self.slot_keys.add(name)
+                for name, shape in (spec.get("int_slots") or {}).items():
+                    entry[name] = torch.zeros((self.max_seqs, *shape), dtype=torch.int32, device=device)
                     self.slot_keys.add(name)
                 self.layers.append(entry)
             elif spec["kind"] == "attention":

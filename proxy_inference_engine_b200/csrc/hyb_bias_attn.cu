@@ -109,7 +109,7 @@ __global__ void __launch_bounds__(kRunWarps * 32) bias_run_kernel(OT* out, const
   float* qs = sm;                       // [d]
   float* mg = qs + d;                   // [warps][dv + 2]: acc, m, l
   float* part = mg + NW * (dv + 2);     // [dv + 2]: this CTA's merged partial softmax
-  for (int c = threadIdx.x; c < d; c += NTH) qs[c] = q[((size_t)t * a.H + h) * d + c];
+  for (int c = threadIdx.x; c < d; c += NTH) qs[c] = q[(size_t)t * a.q_ld + (size_t)h * d + c];
   __syncthreads();
   const int lo = a.window > 0 ? max(0, p - a.window + 1) : 0;
   // this CTA's slice of the keys lo .. p: whole 32-key blocks, in order of rank
@@ -168,7 +168,7 @@ __global__ void __launch_bounds__(kRunWarps * 32) bias_run_kernel(OT* out, const
       for (int u = 0; u < 4; ++u) {
         w[u] = __shfl_sync(0xffffffffu, pj, k0 + u);
         const long long sl = __shfl_sync(0xffffffffu, slot, k0 + u);
-        const KT* vr = vpool + ((size_t)sl * a.G + g) * dv;
+        const KT* vr = vpool + (size_t)sl * a.v_ld + (size_t)g * dv;
 #pragma unroll
         for (int x = 0; x < NV; ++x) {
           const int c = lane + 32 * x;
@@ -276,12 +276,16 @@ __device__ __forceinline__ void cp16(uint32_t dst, const void* src) {
 template <int ROWB>   // bytes of a tile row (>= 128); 16-byte chunk c of row r sits at chunk c ^ (r & 7)
 __device__ __forceinline__ uint32_t tile_off(int r, int c) { return (uint32_t)(r * ROWB + ((c ^ (r & 7)) << 4)); }
 
-template <int D, int DV>
+// SHARED (latent attention): one key / value head whose values are the leading DV features of the key rows, so a key tile
+// is loaded once and serves both products.
+template <int D, int DV, bool SHARED>
 __global__ void __launch_bounds__(128) bias_tile_kernel(__nv_bfloat16* out, const float* q, const float* proj, long long ld,
                                                         const pieh_bias_attn a, const pieh_batch b) {
   constexpr int KC = D / 16, NT = 8, DT = DV / 8;
-  constexpr int KROWB = D * 2, VROWB = DV * 2;
-  constexpr int KTILE = 64 * KROWB, VTILE = 64 * VROWB;
+  constexpr int KROWB = (D * 2 + 127) / 128 * 128;   // the swizzle permutes whole 128-byte runs
+  constexpr int VROWB = SHARED ? KROWB : DV * 2;
+  constexpr int KTILE = 64 * KROWB, VTILE = SHARED ? 0 : 64 * VROWB;
+  static_assert(D % 32 == 0 && DV % 16 == 0 && (SHARED ? DV <= D : DV % 64 == 0), "tile shape");
   extern __shared__ __align__(128) uint8_t smem[];
   pdl_sync();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
@@ -296,20 +300,21 @@ __global__ void __launch_bounds__(128) bias_tile_kernel(__nv_bfloat16* out, cons
   const int32_t* table = b.block_table + (size_t)i * b.bt_stride;
   const __nv_bfloat16* kpool = reinterpret_cast<const __nv_bfloat16*>(a.k_pages);
   const __nv_bfloat16* vpool = reinterpret_cast<const __nv_bfloat16*>(a.v_pages);
-  const uint32_t sK = (uint32_t)__cvta_generic_to_shared(smem), sV = sK + 2 * KTILE;
+  const uint32_t sK = (uint32_t)__cvta_generic_to_shared(smem), sV = SHARED ? sK : sK + 2 * KTILE;
 
   auto issue = [&](int j) {
     const size_t page = (size_t)table[j] * kPage;
     const uint32_t dk = sK + ((j - j_lo) & 1) * KTILE, dvv = sV + ((j - j_lo) & 1) * VTILE;
-    constexpr int CK = KROWB / 16, CV = VROWB / 16;
+    constexpr int CK = D / 8, CV = DV / 8;
     for (int e = tid; e < 64 * CK; e += 128) {
       const int r = e / CK, c = e - r * CK;
       cp16(dk + tile_off<KROWB>(r, c), kpool + ((page + r) * a.G + kvh) * D + c * 8);
     }
-    for (int e = tid; e < 64 * CV; e += 128) {
-      const int r = e / CV, c = e - r * CV;
-      cp16(dvv + tile_off<VROWB>(r, c), vpool + ((page + r) * a.G + kvh) * DV + c * 8);
-    }
+    if (!SHARED)
+      for (int e = tid; e < 64 * CV; e += 128) {
+        const int r = e / CV, c = e - r * CV;
+        cp16(dvv + tile_off<VROWB>(r, c), vpool + (page + r) * a.v_ld + (size_t)kvh * DV + c * 8);
+      }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   issue(j_lo);
@@ -318,8 +323,8 @@ __global__ void __launch_bounds__(128) bias_tile_kernel(__nv_bfloat16* out, cons
   const int r0 = warp * 16 + g, r1 = r0 + 8;
   uint32_t qf[KC][4];
   {
-    const float* q0 = q + ((size_t)(row0 + min(r0, nrows - 1)) * a.H + h) * D;
-    const float* q1 = q + ((size_t)(row0 + min(r1, nrows - 1)) * a.H + h) * D;
+    const float* q0 = q + (size_t)(row0 + min(r0, nrows - 1)) * a.q_ld + (size_t)h * D;
+    const float* q1 = q + (size_t)(row0 + min(r1, nrows - 1)) * a.q_ld + (size_t)h * D;
 #pragma unroll
     for (int kc = 0; kc < KC; ++kc) {
       const float2 x0 = *reinterpret_cast<const float2*>(q0 + kc * 16 + 2 * t4);
@@ -348,7 +353,7 @@ __global__ void __launch_bounds__(128) bias_tile_kernel(__nv_bfloat16* out, cons
     if (j < j_hi) { issue(j + 1); asm volatile("cp.async.wait_group 1;" ::: "memory"); }
     else asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
-    const uint32_t tk = sK + ((j - j_lo) & 1) * KTILE, tv = sV + ((j - j_lo) & 1) * VTILE;
+    const uint32_t tk = sK + ((j - j_lo) & 1) * KTILE, tv = SHARED ? tk : sV + ((j - j_lo) & 1) * VTILE;
     float s[NT][4];
 #pragma unroll
     for (int n = 0; n < NT; ++n) { s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f; }
@@ -451,25 +456,30 @@ __global__ void __launch_bounds__(128) bias_tile_kernel(__nv_bfloat16* out, cons
   }
 }
 
-template <int D, int DV>
+template <int D, int DV, bool SHARED>
 static cudaError_t launch_tile(__nv_bfloat16* out, const float* q, const float* proj, long long ld, const pieh_bias_attn& a,
                                const pieh_batch& b, cudaStream_t st) {
-  constexpr int smem = 2 * (64 * D * 2 + 64 * DV * 2);
+  constexpr int smem = 2 * 64 * ((D * 2 + 127) / 128 * 128 + (SHARED ? 0 : DV * 2));
   static unsigned long long configured = 0;
   int dev = 0;
   cudaGetDevice(&dev);
   if (!(configured >> (dev & 63) & 1)) {
-    cudaError_t e = cudaFuncSetAttribute(bias_tile_kernel<D, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(bias_tile_kernel<D, DV, SHARED>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return e;
     configured |= 1ull << (dev & 63);
   }
-  return launch_k(bias_tile_kernel<D, DV>, dim3(b.n_tiles, a.H), dim3(128), smem, st, out, q, proj, ld, a, b);
+  return launch_k(bias_tile_kernel<D, DV, SHARED>, dim3(b.n_tiles, a.H), dim3(128), smem, st, out, q, proj, ld, a, b);
 }
+
+// one key / value head whose values are the leading features of the cached key rows
+static bool tile_shared(const pieh_bias_attn& a) { return a.G == 1 && a.v_pages == a.k_pages && a.v_ld == a.d; }
 
 // the tile kernel serves steps that are mostly prompt portions, over bf16 pages, at the head sizes it is built for
 static bool tile_ok(const pieh_bias_attn& a, const pieh_batch& b, int out_dtype) {
   static const bool off = [] { const char* e = getenv("PIE_HYBRID_NO_TILE_ATTN"); return e && e[0] == '1'; }();
-  return !off && a.kv_dtype == PIE_DTYPE_BF16 && out_dtype == PIE_DTYPE_BF16 && a.d == a.dv && (a.d == 64 || a.d == 128) &&
+  const bool shape = tile_shared(a) ? (a.dv == 64 || a.dv == 128) && (a.d == a.dv || a.d == a.dv + 32 || a.d == a.dv + 64)
+                                    : a.d == a.dv && (a.d == 64 || a.d == 128) && a.v_ld == (long long)a.G * a.dv;
+  return !off && a.kv_dtype == PIE_DTYPE_BF16 && out_dtype == PIE_DTYPE_BF16 && shape && a.q_ld % 2 == 0 &&
          b.n_tiles > 0 && b.tile_seq && b.tile_row && a.H <= 65535 && (long long)b.T >= 16LL * b.n_seq;
 }
 
@@ -477,7 +487,7 @@ static bool bias_attn_ok(const pieh_bias_attn* a) {
   return a && a->H > 0 && a->G > 0 && a->H % a->G == 0 && a->d > 0 && a->dv > 0 && a->dv <= 512 && a->d <= 1024 &&
          a->k_pages && a->v_pages && a->temp_every >= 0.0 && a->window >= 0 && a->k_off >= 0 && a->v_off >= 0 &&
          a->rot_dims >= 0 && a->rot_dims <= a->d && (a->rot_dims & 1) == 0 && (a->rot_dims == 0 || a->rot_cs) &&
-         (!a->v_mix || a->v_keep) && (a->sigmoid == 0 || a->sigmoid == 1);
+         (!a->v_mix || a->v_keep) && (a->sigmoid == 0 || a->sigmoid == 1) && a->q_ld >= 0 && a->v_ld >= 0;
 }
 
 template <typename KT, typename OT, int NV>
@@ -532,16 +542,24 @@ extern "C" int pieh_bias_attn_prepare(float* q_out, const float* proj, long long
 }
 
 extern "C" int pieh_bias_attn_run(void* out, int out_dtype, const float* q, const float* proj, long long ld,
-                                  const pieh_bias_attn* a, const pieh_batch* b, void* stream) {
-  if (!out || !q || !a || !b || (a->g_off >= 0 && !proj)) return PIE_ENULL;
-  if (!bias_attn_ok(a)) return PIE_EINVAL_SHAPE;
+                                  const pieh_bias_attn* desc, const pieh_batch* b, void* stream) {
+  if (!out || !q || !desc || !b || (desc->g_off >= 0 && !proj)) return PIE_ENULL;
+  if (!bias_attn_ok(desc)) return PIE_EINVAL_SHAPE;
   if (b->T == 0) return PIE_OK;
+  pieh_bias_attn full = *desc;      // with the row strides spelled out
+  if (!full.q_ld) full.q_ld = (long long)full.H * full.d;
+  if (!full.v_ld) full.v_ld = (long long)full.G * full.dv;
+  const pieh_bias_attn* a = &full;
   cudaStream_t st = (cudaStream_t)stream;
   typedef __nv_bfloat16 bf;
   count_launch();
   cudaError_t e;
   if (tile_ok(*a, *b, out_dtype)) {
-    e = a->d == 64 ? launch_tile<64, 64>((bf*)out, q, proj, ld, *a, *b, st) : launch_tile<128, 128>((bf*)out, q, proj, ld, *a, *b, st);
+#define PIEH_TILE(D, DV, SH) launch_tile<D, DV, SH>((bf*)out, q, proj, ld, *a, *b, st)
+    if (!tile_shared(*a)) e = a->d == 64 ? PIEH_TILE(64, 64, false) : PIEH_TILE(128, 128, false);
+    else if (a->dv == 64) e = a->d == 64 ? PIEH_TILE(64, 64, true) : a->d == 96 ? PIEH_TILE(96, 64, true) : PIEH_TILE(128, 64, true);
+    else e = a->d == 128 ? PIEH_TILE(128, 128, true) : a->d == 160 ? PIEH_TILE(160, 128, true) : PIEH_TILE(192, 128, true);
+#undef PIEH_TILE
     return status_of(e);
   }
   if (a->kv_dtype == PIE_DTYPE_BF16)

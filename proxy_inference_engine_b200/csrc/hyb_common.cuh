@@ -110,6 +110,12 @@ __device__ __forceinline__ float xielu_f(float z, float a, float b) {
   return z > 0.f ? fmaf(a * z, z, 0.5f * z) : fmaf(b, expm1f(z) - z, 0.5f * z);
 }
 
+// z / 2 (1 + tanh(u)) = z sigmoid(2 u) with u = sqrt(2 / pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gelu_f(float z) {
+  const float u = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);
+  return z / (1.f + expf(-2.f * u));
+}
+
 // out dtype dispatch for host launchers
 #define PIEH_DISPATCH_DTYPE(code, T, ...)                     \
   do {                                                        \

@@ -23,6 +23,7 @@ __device__ __forceinline__ void lin_store(const LinArgs& a, int m, int n, float 
   else if (a.epi == PIEH_EPI_SOFTCAP) y = a.epi_a * tanhf(y / a.epi_a);
   else if (a.epi == PIEH_EPI_TANH) y = tanhf(y);
   else if (a.epi == PIEH_EPI_XIELU) y = xielu_f(y, a.epi_a, a.epi_b);
+  else if (a.epi == PIEH_EPI_GELU) y = gelu_f(y);
   else if (a.epi == PIEH_EPI_SIGMUL) y *= 1.f / (1.f + expf(-a.gate[(size_t)blockIdx.z * a.gate_bs + (size_t)m * a.gate_ld + n]));
   if (a.epi == PIEH_EPI_STREAMS) {
     float* xs = reinterpret_cast<float*>(a.out) + (size_t)m * a.S * a.N + n;
@@ -141,6 +142,7 @@ __global__ void __launch_bounds__(256) linear_rows_kernel(const LinArgs a) {
   int mb = 0, M = a.M;   // grouped: one slot per blockIdx.y, with its own expert's matrix
   if (a.g_expert) {
     mb = blockIdx.y;
+    if (a.g_expert[mb] < 0) return;   // past the last slot that holds an expert (the whole CTA leaves)
     M = 1;
     w += (size_t)a.g_expert[mb] * a.g_wstride;
     x += (size_t)(a.g_rows ? a.g_rows[mb] : mb) * a.x_ld;
@@ -303,7 +305,9 @@ extern "C" int pieh_linear_act(void* out, int out_dtype, long long out_ld, const
   if (!out || !x || !w) return PIE_ENULL;
   if (M < 0 || N <= 0 || K <= 0) return PIE_EINVAL_SHAPE;
   if (M == 0) return PIE_OK;
-  if (act != PIEH_EPI_NONE && act != PIEH_EPI_RELU2 && act != PIEH_EPI_TANH && act != PIEH_EPI_XIELU) return PIE_EUNSUPPORTED;
+  if (act != PIEH_EPI_NONE && act != PIEH_EPI_RELU2 && act != PIEH_EPI_TANH && act != PIEH_EPI_XIELU &&
+      act != PIEH_EPI_GELU)
+    return PIE_EUNSUPPORTED;
   LinArgs a{out, out_ld, x, x_ld, w, bias, M, N, K, act, act_a, nullptr, nullptr, 0};
   a.epi_b = act_b;
   return run_linear(a, out_dtype, x_dtype, w_dtype, (cudaStream_t)stream);

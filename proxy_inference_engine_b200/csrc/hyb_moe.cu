@@ -1,8 +1,9 @@
 // Mixture-of-experts routing and the plan of the grouped products.
 //   moe_route_kernel   one warp per token.  softmax_top: the largest logits, weights = softmax over the chosen logits.
-//                      Otherwise: sigmoid scores, group scores (sum of a group's two largest), the best groups
-//                      stay eligible, the `top` largest eligible scores are chosen (ties: lower index) with weight
-//                      score * scale; it also counts the tokens of every expert
+//                      Otherwise: scores s (sigmoid, or softmax over all outputs), choice scores s + correction, group scores
+//                      (sum of a group's two largest choice scores, or its largest), the best groups stay eligible, the `top`
+//                      largest eligible choice scores are chosen (ties: lower index) with weight s * scale; it also counts the
+//                      tokens of every expert.  Outputs past the E experts are identity experts: they get no slot
 //   moe_plan_kernel    one CTA: prefix sums of the counts -> every (token, choice) pair gets a SLOT in its expert's run,
 //                      and the runs are cut into tiles of <= 64 and <= 128 slots for the grouped matrix products
 //                      (pieh_moe_linear, hyb_linear.cu).  The order of the pairs inside a run is whatever the atomics
@@ -16,11 +17,12 @@ constexpr int kMaxExperts = 1024, kMaxTop = 32;
 
 __global__ void __launch_bounds__(32) moe_route_kernel(const float* z, long long ld, const pieh_moe_plan p) {
   __shared__ float s[kMaxExperts];
+  __shared__ float ch[kMaxExperts];    // choice scores
   __shared__ float gsc[kMaxExperts];
   __shared__ unsigned char ok[kMaxExperts];   // per group: eligible
   pdl_sync();
   const int t = blockIdx.x, lane = threadIdx.x;
-  const int E = p.E, per = E / p.n_groups;
+  const int E = p.E, N = E + p.identity, per = N / p.n_groups;   // N router outputs
   if (p.softmax_top) {
     // the `top` largest logits, weighted by the softmax over those logits alone (ties: lower index)
     __shared__ float chosen[kMaxTop];
@@ -54,21 +56,31 @@ __global__ void __launch_bounds__(32) moe_route_kernel(const float* z, long long
     }
     return;
   }
-  for (int e = lane; e < E; e += 32) s[e] = 1.f / (1.f + expf(-z[(size_t)t * ld + e]));
+  if (p.softmax_all) {
+    float mx = -INFINITY, sum = 0.f;
+    for (int e = lane; e < N; e += 32) { s[e] = z[(size_t)t * ld + e]; mx = fmaxf(mx, s[e]); }
+    mx = warp_max(mx);
+    for (int e = lane; e < N; e += 32) { s[e] = expf(s[e] - mx); sum += s[e]; }
+    sum = warp_sum(sum);
+    for (int e = lane; e < N; e += 32) s[e] /= sum;
+  } else {
+    for (int e = lane; e < N; e += 32) s[e] = 1.f / (1.f + expf(-z[(size_t)t * ld + e]));
+  }
+  for (int e = lane; e < N; e += 32) ch[e] = p.correction ? s[e] + p.correction[e] : s[e];
   __syncwarp();
   for (int g = lane; g < p.n_groups; g += 32) {
-    float a = -1.f, b = -1.f;   // scores are in (0, 1)
+    float a = -INFINITY, b = -INFINITY;
     for (int e = g * per; e < (g + 1) * per; ++e) {
-      const float v = s[e];
+      const float v = ch[e];
       if (v > a) { b = a; a = v; } else if (v > b) b = v;
     }
-    gsc[g] = per > 1 ? a + b : a;
+    gsc[g] = per > 1 && !p.group_best ? a + b : a;
     ok[g] = 0;
   }
   __syncwarp();
-  // argmax rounds over the warp: value descending, index ascending
+  // argmax rounds over the warp: value descending, index ascending; what is taken or not eligible is at -inf
   auto pick = [&](const float* val, int n, auto usable) {
-    float bv = -2.f;
+    float bv = -INFINITY;
     int bi = n;
     for (int i = lane; i < n; i += 32)
       if (usable(i) && val[i] > bv) { bv = val[i]; bi = i; }
@@ -87,14 +99,14 @@ __global__ void __launch_bounds__(32) moe_route_kernel(const float* z, long long
     __syncwarp();
   }
   for (int r = 0; r < p.top; ++r) {
-    const int e = pick(s, E, [&](int i) { return ok[i / per] == 1 && s[i] >= 0.f; });
+    const int e = pick(ch, N, [&](int i) { return ok[i / per] == 1; });
     __syncwarp();
     if (lane == 0) {
-      const int ee = e < E ? e : 0;   // fewer eligible experts than `top` cannot happen with a valid configuration
-      p.pair_slot[(size_t)t * p.top + r] = ee;            // expert id for now; the plan turns it into a slot
-      p.pair_w[(size_t)t * p.top + r] = e < E ? s[ee] * p.scale : 0.f;
-      atomicAdd(&p.counters[ee], 1);
-      if (e < E) s[ee] = -1.f;                            // taken
+      const int ee = e < N ? e : 0;   // fewer eligible outputs than `top` cannot happen with a valid configuration
+      p.pair_slot[(size_t)t * p.top + r] = ee < E ? ee : -1;   // expert number for now; the plan turns it into a slot
+      p.pair_w[(size_t)t * p.top + r] = e < N ? s[ee] * p.scale : 0.f;
+      if (ee < E) atomicAdd(&p.counters[ee], 1);
+      if (e < N) ch[ee] = -INFINITY;                           // taken
     }
     __syncwarp();
   }
@@ -128,11 +140,13 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const pieh_moe_plan p, i
   }
   for (int q = threadIdx.x; q < P; q += blockDim.x) {
     const int e = p.pair_slot[q];
+    if (e < 0) continue;   // identity expert: no slot
     const int slot = off[e] + atomicAdd(&cur[e], 1);
     p.pair_slot[q] = slot;
     p.slot_row[slot] = q / p.top;
     p.slot_expert[slot] = e;
   }
+  for (int q = off[E] + threadIdx.x; q < P; q += blockDim.x) { p.slot_row[q] = 0; p.slot_expert[q] = -1; }   // unused slots
   __syncthreads();
   for (int e = threadIdx.x; e < E; e += blockDim.x) p.counters[e] = 0;   // ready for the next step
 }
@@ -145,9 +159,10 @@ extern "C" int pieh_moe_route(const float* z, long long ld, const pieh_moe_plan*
   if (!z || !p || !p->slot_row || !p->slot_expert || !p->pair_slot || !p->pair_w || !p->tiles64 || !p->tiles128 ||
       !p->counters)
     return PIE_ENULL;
-  if (T < 0 || p->E < 1 || p->E > kMaxExperts || p->top < 1 || p->top > kMaxTop || p->n_groups < 1 ||
-      p->E % p->n_groups != 0 || p->keep_groups < 1 || p->keep_groups > p->n_groups ||
-      (long long)p->keep_groups * (p->E / p->n_groups) < p->top)
+  if (p->identity < 0 || (p->softmax_top && (p->identity || p->softmax_all))) return PIE_EINVAL_SHAPE;
+  const int n = p->E + p->identity;
+  if (T < 0 || p->E < 1 || n > kMaxExperts || p->top < 1 || p->top > kMaxTop || p->n_groups < 1 || n % p->n_groups != 0 ||
+      p->keep_groups < 1 || p->keep_groups > p->n_groups || (long long)p->keep_groups * (n / p->n_groups) < p->top)
     return PIE_EINVAL_SHAPE;
   if (T == 0) return PIE_OK;
   cudaStream_t st = (cudaStream_t)stream;

@@ -343,6 +343,52 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(OT* cq_out, const f
     elem<KT>::store(pages + slot * kv_rank + c, row[kv_off + c] * ik * kv_norm[c]);
 }
 
+// one CTA per token: the latent's norm and the shared rotated key part -> page; every head's rotated query part
+template <typename QT, typename KT>
+__global__ void __launch_bounds__(256) latent_rot_kernel(const float* proj, long long ld, const pieh_latent_rot a,
+                                                         const pieh_batch b) {
+  __shared__ float red[33];
+  pdl_sync();
+  const int t = blockIdx.x;
+  const int i = b.tok_seq[t], p = b.tok_pos[t];
+  const float* row = proj + (size_t)t * ld;
+  const float* lat = row + a.kv_off;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < a.kv_rank; c += blockDim.x) ss = fmaf(lat[c], lat[c], ss);
+  const float ik = 1.f / sqrtf(block_sum(ss, red) / (float)a.kv_rank + a.eps);
+  const size_t slot = (size_t)b.block_table[(size_t)i * b.bt_stride + p / kPageTokens] * kPageTokens + p % kPageTokens;
+  KT* page = reinterpret_cast<KT*>(a.pages) + slot * (a.kv_rank + a.rot_dim);
+  for (int c = threadIdx.x; c < a.kv_rank; c += blockDim.x) elem<KT>::store(page + c, lat[c] * ik * a.kv_norm[c]);
+  const int half = a.rot_n >> 1, rest = a.rot_dim - a.rot_n, per = half + rest;
+  const float* cs = a.rot_cs ? a.rot_cs + (size_t)t * half * 2 : nullptr;
+  // one work item per rotated pair or passed-through feature: part H is the shared key part, parts 0 .. H - 1 the heads' queries
+  // (a pair is read whole before it is written, so the queries may be rotated where they are)
+  for (int e = threadIdx.x; e < (a.H + 1) * per; e += blockDim.x) {
+    const int h = e / per, f = e - h * per;
+    const float* src = h < a.H ? row + a.q_off + h * a.q_head + a.rot_at : lat + a.kv_rank;
+    float* q = a.q_rot + (size_t)t * a.q_rot_ld + (size_t)(h < a.H ? h : 0) * a.q_rot_head;
+    KT* kd = page + a.kv_rank;
+    if (f < half) {
+      const float u = src[f], v = src[f + half], co = cs[2 * f], si = cs[2 * f + 1];
+      const float x = u * co - v * si, y = v * co + u * si;
+      if (h < a.H) { q[f] = x; q[f + half] = y; }
+      else { elem<KT>::store(kd + f, x); elem<KT>::store(kd + f + half, y); }
+    } else {
+      const int c = a.rot_n + f - half;
+      const float x = src[c];
+      if (h < a.H) q[c] = x; else elem<KT>::store(kd + c, x);
+    }
+  }
+  if (a.q_plain) {
+    QT* qp = reinterpret_cast<QT*>(a.q_plain) + (size_t)t * a.H * a.rot_at;
+    const int n = (int)a.rot_at;
+    for (int e = threadIdx.x; e < a.H * n; e += blockDim.x) {
+      const int h = e / n, f = e - h * n;
+      elem<QT>::store(qp + e, row[a.q_off + h * a.q_head + f]);
+    }
+  }
+}
+
 __global__ void rot_table_kernel(float* cs, const int32_t* positions, const double* freqs, int half, long long n) {
   pdl_sync();
   const long long e = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -451,6 +497,21 @@ extern "C" int pieh_latent_prepare(void* cq_out, int out_dtype, const float* pro
       launch_k(latent_prepare_kernel<OT, KT>, dim3(b->T), dim3(256), 0, (cudaStream_t)stream, (OT*)cq_out, proj, ld, q_rank,
                kv_off, kv_rank, q_norm, kv_norm, eps, (KT*)pages, *b)));
   return status_of(cudaGetLastError());
+}
+
+extern "C" int pieh_latent_rot_prepare(const float* proj, long long ld, const pieh_latent_rot* a, const pieh_batch* b,
+                                       void* stream) {
+  if (!proj || !a || !b || !a->kv_norm || !a->pages || (a->rot_dim > 0 && !a->q_rot) || (a->rot_n > 0 && !a->rot_cs))
+    return PIE_ENULL;
+  if (a->H < 1 || a->kv_rank < 1 || a->rot_dim < 0 || a->rot_n < 0 || a->rot_n > a->rot_dim || (a->rot_n & 1) || a->q_off < 0 ||
+      a->q_head < 0 || a->rot_at < 0 || a->kv_off < 0)
+    return PIE_EINVAL_SHAPE;
+  if (b->T == 0) return PIE_OK;
+  count_launch();
+  cudaError_t e = cudaSuccess;
+  PIEH_DISPATCH_DTYPE(a->q_plain_dtype, QT, PIEH_DISPATCH_DTYPE(a->kv_dtype, KT,
+      e = launch_k(latent_rot_kernel<QT, KT>, dim3(b->T), dim3(256), 0, (cudaStream_t)stream, proj, ld, *a, *b)));
+  return status_of(e);
 }
 
 extern "C" int pieh_rot_table(float* cs, const int32_t* positions, const double* freqs, int T, int half, void* stream) {

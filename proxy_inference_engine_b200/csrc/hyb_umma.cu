@@ -120,6 +120,7 @@ __device__ __forceinline__ void umma_store(const LinArgs& a, int m, int n0, cons
       else if (a.epi == PIEH_EPI_SOFTCAP) t = a.epi_a * tanhf(t / a.epi_a);
       else if (a.epi == PIEH_EPI_TANH) t = tanhf(t);
       else if (a.epi == PIEH_EPI_XIELU) t = xielu_f(t, a.epi_a, a.epi_b);
+      else if (a.epi == PIEH_EPI_GELU) t = gelu_f(t);
       else if (a.epi == PIEH_EPI_SIGMUL && n < a.N) t *= 1.f / (1.f + __expf(-gate[n]));
       y[q] = t;
     }
