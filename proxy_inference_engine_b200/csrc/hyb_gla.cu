@@ -24,38 +24,61 @@ namespace pieh {
 
 namespace cg = cooperative_groups;
 
-__device__ __forceinline__ float root_sigmoid(float z, float inv_tau) { return expf(-softplus_f(-z) * inv_tau); }
+// sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau).  The inner exponential only has to be good to a few ulp: its error reaches
+// the result divided by tau and by 1 + e^z, and e^-z itself is the answer's order below z = -20.
+__device__ __forceinline__ float root_sigmoid(float z, float inv_tau) {
+  const float sp = z < -20.f ? -z : logf(1.f + __expf(-z));
+  return expf(-sp * inv_tau);
+}
 
 // ---- decays ------------------------------------------------------------------------------------------------------------
-constexpr int kDecayRows = 8;
+constexpr int kDecayRows = 16;
 
-// grid (ceil(C / 256), ceil(T / 8)): a thread keeps one channel of 8 rows, so a row of w2t is read once per 8 tokens
+// grid (ceil(C / 64 V), ceil(T / 16)): a thread keeps V neighbouring channels of 4 rows; V = 4 needs C a multiple of 4
+template <int V>
 __global__ void __launch_bounds__(256) gla_decay_kernel(float* decay, const float* proj, long long ld, long long low_off,
                                                         int rank, const float* w2t, const float* bias, float inv_tau, int C,
                                                         int T) {
-  extern __shared__ float low[];   // [8][rank]
+  extern __shared__ __align__(16) float low[];   // [rank][16]
   pdl_sync();
   const int t0 = blockIdx.y * kDecayRows, nr = min(kDecayRows, T - t0);
   for (int e = threadIdx.x; e < kDecayRows * rank; e += blockDim.x) {
     const int r = e / rank, j = e - r * rank;
-    low[e] = r < nr ? proj[(size_t)(t0 + r) * ld + low_off + j] : 0.f;
+    low[j * kDecayRows + r] = r < nr ? proj[(size_t)(t0 + r) * ld + low_off + j] : 0.f;
+  }
+  const int c = (blockIdx.x * 64 + (threadIdx.x & 63)) * V, rg = (threadIdx.x >> 6) * 4;
+  float z[4][V];
+#pragma unroll
+  for (int v = 0; v < V; ++v) {
+    const float b = bias && c + v < C ? bias[c + v] : 0.f;
+#pragma unroll
+    for (int r = 0; r < 4; ++r) z[r][v] = b;
   }
   __syncthreads();
-  const int c = blockIdx.x * blockDim.x + threadIdx.x;
   if (c >= C) return;
-  float z[kDecayRows];
-  const float b = bias ? bias[c] : 0.f;
-#pragma unroll
-  for (int r = 0; r < kDecayRows; ++r) z[r] = b;
-#pragma unroll 4
+#pragma unroll 8
   for (int j = 0; j < rank; ++j) {
-    const float w = w2t[(size_t)j * C + c];
+    float w[V];
+    if (V == 4) {
+      const float4 x = *reinterpret_cast<const float4*>(w2t + (size_t)j * C + c);
+      w[0] = x.x; w[1 % V] = x.y; w[2 % V] = x.z; w[3 % V] = x.w;
+    } else w[0] = w2t[(size_t)j * C + c];
+    const float4 l = *reinterpret_cast<const float4*>(low + j * kDecayRows + rg);
+    const float lr[4] = {l.x, l.y, l.z, l.w};
 #pragma unroll
-    for (int r = 0; r < kDecayRows; ++r) z[r] = fmaf(w, low[r * rank + j], z[r]);
+    for (int r = 0; r < 4; ++r)
+#pragma unroll
+      for (int v = 0; v < V; ++v) z[r][v] = fmaf(w[v], lr[r], z[r][v]);
   }
 #pragma unroll
-  for (int r = 0; r < kDecayRows; ++r)
-    if (r < nr) decay[(size_t)(t0 + r) * C + c] = root_sigmoid(z[r], inv_tau);
+  for (int r = 0; r < 4; ++r) {
+    if (rg + r >= nr) break;
+    float* dst = decay + (size_t)(t0 + rg + r) * C + c;
+    if (V == 4)
+      *reinterpret_cast<float4*>(dst) = make_float4(root_sigmoid(z[r][0], inv_tau), root_sigmoid(z[r][1 % V], inv_tau),
+                                                    root_sigmoid(z[r][2 % V], inv_tau), root_sigmoid(z[r][3 % V], inv_tau));
+    else dst[0] = root_sigmoid(z[r][0], inv_tau);
+  }
 }
 
 // ---- the scan ----------------------------------------------------------------------------------------------------------
@@ -372,16 +395,25 @@ __global__ void __launch_bounds__(256) gla_step_kernel(OT* out, const float* pro
   }
   for (int c = threadIdx.x; c < g.rank; c += 256) low[c] = row[g.low_off + c];
   __syncthreads();
-  for (int c = threadIdx.x; c < dk; c += 256) {
-    const size_t C = (size_t)d.H * dk, ch = (size_t)h * dk + c;
-    float z = g.bias ? g.bias[ch] : 0.f;
-#pragma unroll 8
-    for (int r = 0; r < g.rank; ++r) z = fmaf(g.w2t[r * C + ch], low[r], z);
-    as[c] = root_sigmoid(z, g.inv_tau);
-  }
   float v[4];
 #pragma unroll
   for (int e = 0; e < 4; ++e) v[e] = j + e < dv ? row[d.v_off + (size_t)h * dv + j + e] : 0.f;
+  // decay logits: `cuts` threads share a channel's low-rank sum where the head is narrower than the CTA
+  const int cuts = dk <= 64 ? 4 : dk <= 128 ? 2 : 1, span = 256 / cuts;
+  const size_t C = (size_t)d.H * dk;
+  for (int c = threadIdx.x % span; c < dk; c += span) {
+    const size_t ch = (size_t)h * dk + c;
+    float z = 0.f;
+#pragma unroll 16
+    for (int r = threadIdx.x / span; r < g.rank; r += cuts) z = fmaf(g.w2t[r * C + ch], low[r], z);
+    part[(threadIdx.x / span) * dk + c] = z;       // cuts * dk <= 512 floats
+  }
+  __syncthreads();
+  for (int c = threadIdx.x; c < dk; c += 256) {
+    float z = g.bias ? g.bias[(size_t)h * dk + c] : 0.f;
+    for (int k = 0; k < cuts; ++k) z += part[k * dk + c];
+    as[c] = root_sigmoid(z, g.inv_tau);
+  }
   __syncthreads();
   float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
   for (int r0 = rg; r0 < dk; r0 += UN * RG) {
@@ -477,10 +509,16 @@ extern "C" int pieh_gla_decay(float* decay, const float* proj, long long ld, lon
   if (!decay || !proj || !w2t) return PIE_ENULL;
   if (T < 0 || C < 1 || rank < 1 || rank > 1024 || low_off < 0 || !(inv_tau > 0.f)) return PIE_EINVAL_SHAPE;
   if (T == 0) return PIE_OK;
+  const size_t smem = (size_t)kDecayRows * rank * 4;   // at most 64 KB
+  const bool vec = C % 4 == 0 && ((reinterpret_cast<uintptr_t>(decay) | reinterpret_cast<uintptr_t>(w2t)) & 15) == 0;
+  auto kernel = vec ? gla_decay_kernel<4> : gla_decay_kernel<1>;
+  const int per = vec ? 256 : 64;
+  cudaError_t e = cudaSuccess;
+  if (smem > 48 * 1024) e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  if (e != cudaSuccess) return status_of(e);
   count_launch();
-  return status_of(launch_k(gla_decay_kernel, dim3((C + 255) / 256, (T + kDecayRows - 1) / kDecayRows), dim3(256),
-                            (size_t)kDecayRows * rank * 4, (cudaStream_t)stream, decay, proj, ld, low_off, rank, w2t, bias,
-                            inv_tau, C, T));
+  return status_of(launch_k(kernel, dim3((C + per - 1) / per, (T + kDecayRows - 1) / kDecayRows), dim3(256), smem,
+                            (cudaStream_t)stream, decay, proj, ld, low_off, rank, w2t, bias, inv_tau, C, T));
 }
 
 extern "C" int pieh_gla_scan(float* o, const float* proj, long long ld, const float* decay, const pieh_gla* d,

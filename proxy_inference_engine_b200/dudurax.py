@@ -406,7 +406,7 @@ def random_weights(args: DuduraxArgs, seed: int = 0, device="cpu") -> dict:
         w[p + "norm1"] = (1 + 0.2 * rnd(W)).to(bf)
         if cfg["type"] in GLA:
             H, n, dv = m["heads"], m["dim"], m["vdim"]
-            low = max(4, min(64, W // 16))
+            low = max(4, min(16, W // 8))
             w[q + "q"], w[q + "k"], w[q + "v"] = lin(H * n, W, 2.0), lin(H * n, W, 2.0), lin(H * dv, W, 2.0)
             w[q + "g"], w[q + "o"] = lin(H * dv, W, 2.0), lin(W, H * dv, 2.0)
             w[q + "a1"], w[q + "a2"], w[q + "a2.b"] = lin(low, W, 2.0), lin(H * n, low, 2.0), (3 * rnd(H * n)).to(bf)

@@ -1,9 +1,10 @@
-"""Throughput of the Golitar, Babodra, Maginex and Zelinex families at layer sizes of real models (random weights), with
+"""Throughput of the Golitar, Babodra, Maginex, Zelinex and Dudurax families at layer sizes of real models (random weights), with
 every operator of the step timed in place and set against its roofline.  Golitar is shown beside the quantized Llama path
 at equal width / feed-forward / depth; Babodra beside Golitar, Maginex beside Babodra, and Zelinex beside Golitar (the other
-family built on a matrix-state recurrence and windowed attention), at equal width / depth / active feed-forward size.
+family built on a matrix-state recurrence and windowed attention), Dudurax beside Maginex (latent attention, recurrence,
+experts in every layer) and Zelinex (matrix-state scans), at equal width / depth / active feed-forward size.
 
-``run(size, ...)`` is what ``bench.py --family golitar|babodra|maginex|zelinex`` prints.  Method: one prompt of ``prompt`` tokens goes through
+``run(size, ...)`` is what ``bench.py --family golitar|babodra|maginex|zelinex|dudurax`` prints.  Method: one prompt of ``prompt`` tokens goes through
 ``HybridEngine.forward`` in portions of ``portion`` rows (prefill tok/s, CUDA events around all portions), then ``batch``
 sequences decode ``steps`` tokens each (decode tok/s).  The per-operator table wraps every library call of one prefill
 portion and one decode step in a CUDA event pair; bytes and flops are the algorithmic ones of the call's shapes, the
@@ -27,6 +28,9 @@ SIZES = {
                zel=dict(pattern="gpgpgpgpgpgp", loop=(0, 4, 2), d_heads=16, d_dim=128, heads=16, kv_heads=4, dim=128, vdim=128,
                         window=1024, rot_dims=64, s_heads=32, s_vdim=64, state=128, groups=2, norm_groups=2, conv=4,
                         experts=16, top=4, expert_ff=1536, shared_ff=2048),
+               dud=dict(pattern="ggahggahggahggah", gla=(8, 128, 256), gla_2=(4, 256, 512), tau=16.0, heads=16, dim=128,
+                        rot_dim=64, vdim=128, kv_rank=128, window=1024, experts=16, identity=4, groups=(4, 3), top=4,
+                        expert_ff=2048),
                llama=dict(hidden_size=2048, intermediate_size=8192, num_attention_heads=32,
                                                        num_key_value_heads=8, head_dim=64, vocab_size=32000)),
     "8b": dict(width=4096, ff=14336, vocab=32000, pattern="dddadddA", dH=32, dG=16, dk=128, dv=128, aH=32, aG=8, ad=64,
@@ -37,6 +41,9 @@ SIZES = {
                zel=dict(pattern="gpgpgp", loop=(0, 2, 2), d_heads=32, d_dim=128, heads=32, kv_heads=8, dim=128, vdim=128,
                         window=2048, rot_dims=64, s_heads=64, s_vdim=64, state=128, groups=2, norm_groups=2, conv=4,
                         experts=16, top=4, expert_ff=3072, shared_ff=2048),
+               dud=dict(pattern="ggahggah", gla=(16, 128, 256), gla_2=(8, 256, 512), tau=16.0, heads=32, dim=128,
+                        rot_dim=64, vdim=128, kv_rank=128, window=2048, experts=16, identity=4, groups=(4, 3), top=4,
+                        expert_ff=3584),
                llama=dict(hidden_size=4096, intermediate_size=14336, num_attention_heads=32,
                                                 num_key_value_heads=8, head_dim=128, vocab_size=32000)),
 }
@@ -118,6 +125,25 @@ def zelinex_config(size: str) -> dict:
             "loop": {"start": a, "stop": b, "times": t}, "layers": layers}
 
 
+def dudurax_config(size: str) -> dict:
+    """Same width and depth as the others; gated linear attention (two head layouts of key width W / 2 and value width W) and
+    windowed latent attention; the first layer's feed-forward is dense, the others' a mixture with the ACTIVE size of
+    babodra_config's when no identity expert is chosen."""
+    s = SIZES[size]
+    d = s["dud"]
+    gla = lambda hd: {"heads": hd[0], "dim": hd[1], "vdim": hd[2], "tau": d["tau"]}
+    lat = {"heads": d["heads"], "dim": d["dim"], "rot_dim": d["rot_dim"], "vdim": d["vdim"], "kv_rank": d["kv_rank"],
+           "scale": (d["dim"] + d["rot_dim"]) ** -0.5, "mask": {"size": d["window"]}, "rot": {"base": 5e4, "dims": d["rot_dim"]}}
+    moe = {"kind": "moe", "expert": {"ff": d["expert_ff"], "limit": 7.0},
+           "router": {"experts": d["experts"], "identity": d["identity"], "top": d["top"], "scale": 2.0,
+                      "groups": {"count": d["groups"][0], "keep": d["groups"][1]}}}
+    mixers = {"g": ("gla", gla(d["gla"])), "h": ("gla_2", gla(d["gla_2"])), "a": ("latent_attention", lat)}
+    layers = [{"type": mixers[ch][0], "mixer": dict(mixers[ch][1]), "mlp": dict(moe) if i else {"kind": "dense", "ff": s["ff"]}}
+              for i, ch in enumerate(d["pattern"])]
+    return {"architecture": "Dudurax", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5}, "postln_alpha": 2.5,
+            "embedding": {"scale": 4.0, "bigram": {"buckets": 32749, "mul_prev": 31, "mul_cur": 7}}, "layers": layers}
+
+
 def _peaks(root):
     try:
         with open(os.path.join(root, "MEASURED_PEAKS.json")) as f:
@@ -167,6 +193,7 @@ def _cost(name, a, model, batch_info):
         return N * K * wb + M * K * act + M * (N // 2) * ob, 2.0 * M * N * K, f"linear_glu M={M}"
     if name == "pieh_moe_linear":
         P, N, K, glu, E = a[9], a[10], a[11], a[13], a[17]._obj.E
+        P = round(P * E / (E + a[17]._obj.identity))      # identity experts take no product; choices spread evenly on average
         ob = 4 if a[1] == 1 else 2
         wb = 4 if a[7] == 1 else 2
         return min(E, P) * N * K * wb + P * K * act + P * (N // 2 if glu else N) * ob, 2.0 * P * N * K, f"moe_linear P={P}"
@@ -203,6 +230,28 @@ def _cost(name, a, model, batch_info):
             return T * (2 * Cn + 3 * sd.H) * 4, 2.0 * T * Cn * sd.taps, "ssd_prepare"
         return (n_seq * 2 * sd.H * sd.N * sd.P * 4 + T * (Cn + sd.H * sd.P + 2 * sd.H) * 4, 5.0 * T * sd.H * sd.N * sd.P,
                 "ssd_scan")
+    if name == "pieh_sum_norm":
+        Tn, W, mix = a[8], a[9], a[4]
+        parts = mix._obj.top if mix is not None else 1
+        if mix is not None and getattr(model.args, "bigram", None) is not None:     # identity experts read no row
+            r = next(ly["mlp"] for ly in model.layers if ly["mlp"] and ly["mlp"]["kind"] == "moe")
+            parts = parts * r["E"] / (r["E"] + r["identity"])
+        return Tn * W * (4 * parts + 8 + (act if a[1] is not None else 0)), 0.0, "sum_norm" + ("(mixture)" if mix is not None else "")
+    if name == "pieh_embed_pairs":
+        return T * a[12] * (2 * act + 4 + (act if a[1] is not None else 0)), 0.0, "embed"
+    if name == "pieh_gla_decay":
+        return T * (a[8] + a[4]) * 4, 2.0 * T * a[8] * a[4], "gla_decay"
+    if name == "pieh_gla_scan":
+        d = a[4]._obj
+        return (n_seq * 2 * d.H * d.dk * d.dv * 4 + T * d.H * (3 * d.dk + 2 * d.dv) * 4, 5.0 * T * d.H * d.dk * d.dv,
+                "gla_scan")
+    if name == "pieh_gla_step":
+        d = a[12]._obj
+        return (n_seq * 2 * d.H * d.dk * d.dv * 4 + T * d.H * (2 * d.dk + 2 * d.dv) * 4 + a[5] * d.H * d.dk * 4
+                + T * d.H * d.dv * act, 5.0 * T * d.H * d.dk * d.dv, "gla_step")
+    if name == "pieh_latent_rot_prepare":
+        lr = a[2]._obj
+        return T * (lr.kv_rank + lr.rot_dim) * (4 + act) + T * lr.H * lr.rot_dim * 8, 0.0, "latent_rot_prepare"
     if name == "pieh_canon_conv":
         cn = a[0]._obj
         return T * a[3] * (4 + cn.n_out * act), 2.0 * T * a[3] * cn.n_out * cn.taps, "canon_conv"
@@ -233,7 +282,7 @@ def _cost(name, a, model, batch_info):
             per_q = min(per_q, at.window)
             keys = min(keys, at.window + own)
         shared_kv = 1 if at.k_pages == at.v_pages else 2      # latent attention: keys and values are one pool
-        kvb = n_seq * keys * G * (d + dv) * act // (2 if shared_kv == 1 else 1)
+        kvb = n_seq * keys * G * (d if shared_kv == 1 else d + dv) * act
         return (kvb + T * H * (d * 4 + dv * (act + 4)), 2.0 * T * H * per_q * (d + dv),
                 "attn_run" + (f"(window {at.window})" if at.window else "") + ("(latent)" if shared_kv == 1 else ""))
     if name in ("pieh_stream_norm",):
@@ -283,7 +332,16 @@ def run(size="1b", prompt=4096, portion=4096, batch=4, steps=32, warmup=3, root=
 
     hbm, tfl, src = _peaks(root)
     t0 = time.time()
-    if family == "zelinex":
+    if family == "dudurax":
+        from .dudurax import DuduraxArgs, DuduraxModel, random_weights
+        cfg = dudurax_config(size)
+        args = DuduraxArgs.from_dict(cfg)
+        weights = random_weights(args, seed=0, device="cuda")
+        n_params = sum(v.numel() for v in weights.values())
+        model = DuduraxModel(args, weights, "cuda", "bfloat16")
+        del weights
+        pattern = SIZES[size]["dud"]["pattern"]
+    elif family == "zelinex":
         from .zelinex import ZelinexArgs, ZelinexModel, random_weights
         cfg = zelinex_config(size)
         args = ZelinexArgs.from_dict(cfg)
@@ -371,7 +429,11 @@ def run(size="1b", prompt=4096, portion=4096, batch=4, steps=32, warmup=3, root=
            "pipeline_error": int(timed._lib.pieh_pipeline_error()), "setup_s": round(time.time() - t0, 1)}
     del eng, model
     torch.cuda.empty_cache()
-    if family == "zelinex":
+    if family == "dudurax":
+        if with_llama:      # the closest models of the framework at the same sizes: latent attention, recurrence and experts in
+            for other in ("maginex", "zelinex"):                 # every layer; matrix-state scans
+                out[f"{other}_equal_size"] = run(size, prompt, portion, batch, steps, warmup, root, with_llama=False, family=other)
+    elif family == "zelinex":
         if with_llama:      # the closest model of the framework (matrix-state recurrence + windowed attention) at the same sizes
             out["golitar_equal_size"] = run(size, prompt, portion, batch, steps, warmup, root, with_llama=False)
     elif family == "maginex":
