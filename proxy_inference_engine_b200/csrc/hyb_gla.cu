@@ -330,17 +330,24 @@ __global__ void __launch_bounds__(256) gla_carry_kernel(const pieh_gla d, const 
   const int nseg = (len + span - 1) / span;
   const size_t row = e / d.dv, rows = (size_t)d.H * d.dk;
   float carry = b.seq_ctx[i] > 0 ? d.state[(size_t)b.seq_slot[i] * whole + e] : 0.f;
-  size_t seg = (size_t)(tile / sg.tiles + i);
-  float own = sg.states[seg * whole + e], a = sg.decays[seg * rows + row];
-  for (int m = 0; m < nseg; ++m, ++seg) {
-    float own_n = 0.f, a_n = 0.f;
-    if (m + 2 < nseg) {           // the next segment's pair is on its way before this one's state is replaced
-      own_n = sg.states[(seg + 1) * whole + e];
-      a_n = sg.decays[(seg + 1) * rows + row];
+  const size_t seg = (size_t)(tile / sg.tiles + i);
+  constexpr int AHEAD = 8;      // loads in flight: the chain itself is one multiply-add per segment
+  for (int m0 = 0; m0 < nseg; m0 += AHEAD) {
+    float own[AHEAD], a[AHEAD];
+#pragma unroll
+    for (int u = 0; u < AHEAD; ++u) {
+      own[u] = a[u] = 0.f;
+      if (m0 + u + 1 < nseg) {  // nothing follows a sequence's last segment: it has no (A, B)
+        own[u] = sg.states[(seg + m0 + u) * whole + e];
+        a[u] = sg.decays[(seg + m0 + u) * rows + row];
+      }
     }
-    sg.states[seg * whole + e] = carry;
-    carry = fmaf(a, carry, own);
-    own = own_n; a = a_n;
+#pragma unroll
+    for (int u = 0; u < AHEAD; ++u)
+      if (m0 + u < nseg) {
+        sg.states[(seg + m0 + u) * whole + e] = carry;
+        carry = fmaf(a[u], carry, own[u]);
+      }
   }
 }
 
