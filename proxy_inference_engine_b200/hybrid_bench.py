@@ -29,7 +29,7 @@ SIZES = {
                         window=1024, rot_dims=64, s_heads=32, s_vdim=64, state=128, groups=2, norm_groups=2, conv=4,
                         experts=16, top=4, expert_ff=1536, shared_ff=2048),
                dud=dict(pattern="ggahggahggahggah", gla=(8, 128, 256), gla_2=(4, 256, 512), tau=16.0, heads=16, dim=128,
-                        rot_dim=64, vdim=128, kv_rank=128, window=1024, experts=16, identity=4, groups=(4, 3), top=4,
+                        rot_dim=64, vdim=128, kv_rank=128, window=1024, experts=16, identity=4, groups=(5, 3), top=4,
                         expert_ff=2048),
                llama=dict(hidden_size=2048, intermediate_size=8192, num_attention_heads=32,
                                                        num_key_value_heads=8, head_dim=64, vocab_size=32000)),
@@ -42,7 +42,7 @@ SIZES = {
                         window=2048, rot_dims=64, s_heads=64, s_vdim=64, state=128, groups=2, norm_groups=2, conv=4,
                         experts=16, top=4, expert_ff=3072, shared_ff=2048),
                dud=dict(pattern="ggahggah", gla=(16, 128, 256), gla_2=(8, 256, 512), tau=16.0, heads=32, dim=128,
-                        rot_dim=64, vdim=128, kv_rank=128, window=2048, experts=16, identity=4, groups=(4, 3), top=4,
+                        rot_dim=64, vdim=128, kv_rank=128, window=2048, experts=16, identity=4, groups=(5, 3), top=4,
                         expert_ff=3584),
                llama=dict(hidden_size=4096, intermediate_size=14336, num_attention_heads=32,
                                                 num_key_value_heads=8, head_dim=128, vocab_size=32000)),
@@ -133,15 +133,15 @@ def dudurax_config(size: str) -> dict:
     d = s["dud"]
     gla = lambda hd: {"heads": hd[0], "dim": hd[1], "vdim": hd[2], "tau": d["tau"]}
     lat = {"heads": d["heads"], "dim": d["dim"], "rot_dim": d["rot_dim"], "vdim": d["vdim"], "kv_rank": d["kv_rank"],
-           "scale": (d["dim"] + d["rot_dim"]) ** -0.5, "mask": {"size": d["window"]}, "rot": {"base": 5e4, "dims": d["rot_dim"]}}
+           "scale": (d["dim"] + d["rot_dim"]) ** -0.5, "mask": {"size": d["window"]}, "rot": {"base": 1e5, "dims": d["rot_dim"]}}
     moe = {"kind": "moe", "expert": {"ff": d["expert_ff"], "limit": 7.0},
-           "router": {"experts": d["experts"], "identity": d["identity"], "top": d["top"], "scale": 2.0,
+           "router": {"experts": d["experts"], "identity": d["identity"], "top": d["top"], "scale": 1.5,
                       "groups": {"count": d["groups"][0], "keep": d["groups"][1]}}}
     mixers = {"g": ("gla", gla(d["gla"])), "h": ("gla_2", gla(d["gla_2"])), "a": ("latent_attention", lat)}
     layers = [{"type": mixers[ch][0], "mixer": dict(mixers[ch][1]), "mlp": dict(moe) if i else {"kind": "dense", "ff": s["ff"]}}
               for i, ch in enumerate(d["pattern"])]
-    return {"architecture": "Dudurax", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5}, "postln_alpha": 2.5,
-            "embedding": {"scale": 4.0, "bigram": {"buckets": 32749, "mul_prev": 31, "mul_cur": 7}}, "layers": layers}
+    return {"architecture": "Dudurax", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5}, "postln_alpha": 2.0,
+            "embedding": {"scale": 4.0, "bigram": {"buckets": 32749, "mul_prev": 1009, "mul_cur": 37}}, "layers": layers}
 
 
 def _peaks(root):
