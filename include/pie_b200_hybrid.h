@@ -149,6 +149,10 @@ int pieh_attn_run(void* out, int out_dtype, const float* q, const pieh_attn* a, 
 int pieh_linear_glu(void* out, int out_dtype, long long out_ld, const void* x, int x_dtype, long long x_ld, const void* w,
                     int w_dtype, int M, int N, int K, float alpha, float limit, float up_offset, void* stream);
 
+/* The same pair with a choice of gate: act NONE silu(g') * (u' + up_offset), act GELU gelu_tanh(g') * (u' + up_offset). */
+int pieh_linear_glu_act(void* out, int out_dtype, long long out_ld, const void* x, int x_dtype, long long x_ld, const void* w,
+                        int w_dtype, int M, int N, int K, int act, float limit, float up_offset, void* stream);
+
 /* ---- learned absolute positions and the post-norm residual ----------------------------------------------------------
  * x[t, :] = table[tokens[t], :] + pos_table[positions[t], :] (fp32), act[t, :] = the same rounded to the act dtype
  * (act may be NULL).  pos_table NULL: no position term. */
@@ -177,7 +181,7 @@ int pieh_postnorm_add(float* x, void* act, int act_dtype, const float* y, const 
  * projected keys), gate logits at g_off (H dv; g_off < 0: no gate).
  *   q' = rms_norm(q over all H d features) * q_norm * (1 + temp_coef * ln(floor((p + 1) / temp_every) + 1))
  *   k' = rms_norm(k over all G d features) * k_norm            (q_norm / k_norm NULL: no norm; temp_every 0: no factor)
- *   s_ij = q'_i . k'_j * scale - slopes[h] * (i - j),   j <= i  (and i - j < window when window > 0)
+ *   s_ij = q'_i . k'_j * scale - slopes[h] * (i - j),   j <= i  (and, when window > 0, i - j < window or j < keep_first)
  *   p_ij = exp(s_ij) / (sink + sum_j exp(s_ij))                 (sink 1: one extra term of score 0 without a value)
  *   out[i, h, :] = sum_j p_ij v_j * sigmoid(gate[i, h, :]) */
 typedef struct pieh_bias_attn {
@@ -209,6 +213,9 @@ typedef struct pieh_bias_attn {
   long long q_ld;          /* floats between two tokens' queries in pieh_bias_attn_run (0: H d) */
   long long v_ld;          /* elements between two positions' value rows (0: G dv).  With G = 1 and v_pages == k_pages, v_ld = d:
                               the values are the leading dv features of the cached key rows (latent attention) */
+  int keep_first;          /* with a window: the keys at positions < keep_first stay visible (at their true positions) */
+  int head_norm;           /* 1: q_norm / k_norm are [d], every head is normed by its own root mean square */
+  int rot_pairs;           /* 1: features 2 i and 2 i + 1 rotate together instead of i and i + rot_dims / 2 (head_norm 1, or no norms) */
 } pieh_bias_attn;
 /* q_out fp32 [T, H, d]; k' and v appended to the pages at each row's position.  Rotation (after the norms) turns the pair
  * (u, v) = (x[i], x[i + rot_dims / 2]) into (u cos - v sin, v cos + u sin). */
@@ -306,6 +313,15 @@ int pieh_sandwich_add(float* x, const float* y, const pieh_mix_sum* mix, const f
                       const float* add_rows, const float* add_vec, void* h, int h_dtype, const float* next_w, float eps,
                       int T, int W, void* stream);
 
+/* ---- the sandwich with layer norms: ln(v; w, b) = (v - mean) / sqrt(mean((v - mean)^2) + eps) * w + b --------------------------
+ *   post_w set:   x[t, :] += ln(y[t, :]; post_w, post_b)          post_w NULL, y set:  x[t, :] = y[t, :]      (y fp32, stride y_ld)
+ *   x[t, :] += add_rows[t, :] + add_vec[:]                        each optional (rows' stride add_ld; stride 0: W)
+ *   h[r, :] = next_w ? ln(x[t, :]; next_w, next_b) : x[t, :]      act dtype [n, W]; skipped when h is NULL
+ * rows NULL: t = r, n rows, x is updated.  rows given: t = rows[r], only h is written (rows may repeat). */
+int pieh_layernorm_add(float* x, const float* y, long long y_ld, const float* post_w, const float* post_b,
+                       const float* add_rows, long long add_ld, const float* add_vec, void* h, int h_dtype,
+                       const float* next_w, const float* next_b, const int32_t* rows, float eps, int n, int W, void* stream);
+
 /* ---- post-norm residual whose norm REPLACES it, and the pair embedding --------------------------------------------------------
  *   s = alpha * x[t, :] + (y ? y[t, :] : mixture),   x[t, :] = s / sqrt(mean(s^2) + eps) * norm_w,   act[t, :] = x[t, :]
  * The mixture is that of pieh_postnorm_add (a NULL shared_gate: the shared rows count fully), except that part_row < 0 stands
@@ -363,6 +379,7 @@ typedef struct pieh_latent_rot {
   int q_plain_dtype;
   void* pages;
   int kv_dtype;
+  int rot_pairs;           /* 1: features 2 i and 2 i + 1 rotate together */
 } pieh_latent_rot;
 int pieh_latent_rot_prepare(const float* proj, long long ld, const pieh_latent_rot* a, const pieh_batch* b, void* stream);
 

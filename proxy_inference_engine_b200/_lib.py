@@ -169,7 +169,8 @@ class HybBiasAttn(C.Structure):
                 # optional pieces, zero / NULL = off
                 ("sinks", C.c_void_p), ("gate_heads", C.c_int), ("rot_dims", C.c_int), ("rot_cs", C.c_void_p),
                 ("v_mix", C.c_void_p), ("v_keep", C.c_void_p), ("sigmoid", C.c_int), ("score_bias", C.c_void_p),
-                ("q_ld", C.c_longlong), ("v_ld", C.c_longlong)]
+                ("q_ld", C.c_longlong), ("v_ld", C.c_longlong), ("keep_first", C.c_int), ("head_norm", C.c_int),
+                ("rot_pairs", C.c_int)]
 
 
 class HybMixSum(C.Structure):
@@ -219,7 +220,7 @@ class HybLatentRot(C.Structure):
                 ("q_head", C.c_longlong), ("rot_at", C.c_longlong), ("kv_off", C.c_longlong), ("kv_norm", C.c_void_p),
                 ("eps", C.c_float), ("rot_cs", C.c_void_p), ("q_rot", C.c_void_p), ("q_rot_ld", C.c_longlong),
                 ("q_rot_head", C.c_longlong), ("q_plain", C.c_void_p), ("q_plain_dtype", C.c_int), ("pages", C.c_void_p),
-                ("kv_dtype", C.c_int)]
+                ("kv_dtype", C.c_int), ("rot_pairs", C.c_int)]
 
 
 _PB, _PD, _PA = C.POINTER(HybBatch), C.POINTER(HybDelta), C.POINTER(HybAttn)
@@ -268,6 +269,8 @@ HYBRID_SIGNATURES = {
     "pieh_gla_scan": (_i, [_vp, _vp, _ll, _vp, _PGL, _PB, _vp, _i, _vp]),
     "pieh_gla_step": (_i, [_vp, _i, _vp, _ll, _ll, _i, _vp, _vp, _f, _ll, _vp, _f, _PGL, _PB, _vp]),
     "pieh_latent_rot_prepare": (_i, [_vp, _ll, _PLR, _PB, _vp]),
+    "pieh_layernorm_add": (_i, [_vp, _vp, _ll, _vp, _vp, _vp, _ll, _vp, _vp, _i, _vp, _vp, _vp, _f, _i, _i, _vp]),
+    "pieh_linear_glu_act": (_i, [_vp, _i, _ll, _vp, _i, _ll, _vp, _i, _i, _i, _i, _i, _f, _f, _vp]),
     "pieh_moe_route": (_i, [_vp, _ll, _PMP, _i, _vp]),
     "pieh_moe_linear": (_i, [_vp, _i, _ll, _vp, _i, _ll, _vp, _i, _ll, _i, _i, _i, _i, _i, _f, _f, _f, _PMP, _vp]),
 }

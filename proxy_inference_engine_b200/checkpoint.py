@@ -262,10 +262,15 @@ def _load_dudurax(config: dict, path: str, device, dtype):
     return DuduraxModel(DuduraxArgs.from_dict(config), read_weights(path), device, dtype or "bfloat16")
 
 
+def _load_vokusun(config: dict, path: str, device, dtype):
+    from .vokusun import VokusunArgs, VokusunModel
+    return VokusunModel(VokusunArgs.from_dict(config), read_weights(path), device, dtype or "bfloat16")
+
+
 # model registry: config.json's "architecture" (or, for Hugging Face / MLX checkpoints, "model_type") -> loader.
 # The reference resolves model_type to a module of PIE/models/ the same way (PIE/models/utils.py:25-48).
 MODEL_REGISTRY = {"llama": _load_llama, "Golitar": _load_golitar, "Babodra": _load_babodra, "Maginex": _load_maginex,
-                  "Zelinex": _load_zelinex, "Dudurax": _load_dudurax}
+                  "Zelinex": _load_zelinex, "Dudurax": _load_dudurax, "Vokusun": _load_vokusun}
 
 
 def model_kind(config: dict) -> str:

@@ -1,11 +1,12 @@
 // Attention with a per-head linear distance bias, a softmax sink and a sigmoid output gate over 64-token pages, ragged steps.
-//   s_ij = q_i . k_j * scale - slope_h (i - j),  j <= i (and i - j < window if one is set)
+//   s_ij = q_i . k_j * scale - slope_h (i - j),  j <= i (and i - j < window, or j < keep_first, if a window is set)
 //   p_ij = exp(s_ij) / (sink + sum_j exp(s_ij))          sink = 1: a term of score 0 that carries no value, so a query
 //                                                        that matches nothing returns (almost) nothing
 //   out_i = sum_j p_ij v_j * sigmoid(gate_i)
 // Optional: a LEARNED sink logit per head in place of the score-0 sink, one gate logit per head in place of one per
 // feature, a rotation of the leading features of every query / key head ("rotate half" pairing) from a per-step (cos, sin)
-// table, and values blended with another layer's values of the same token before they are cached.
+// table (bias_prepare_heads_kernel: also adjacent features, and a norm per head), and values blended with another layer's
+// values of the same token before they are cached.
 // bias_prepare_kernel   per token: ONE rms norm over all heads' query features (and one over all key features) with
 //                       per-feature weights, the query temperature 1 + c ln(floor((p + 1) / every) + 1), then the normed
 //                       keys go to the key pages and the values -- here usually the PROJECTED keys themselves, v_off ==
@@ -76,6 +77,60 @@ __global__ void __launch_bounds__(256) bias_prepare_kernel(float* q_out, const f
   }
 }
 
+// The per-head form (norm over each head's d features, weight shared by the heads; either rotation pairing): a warp per (token,
+// head), the first H of a token's H + 2 G warps query heads, then key heads, then value heads.
+template <typename KT>
+__global__ void __launch_bounds__(256) bias_prepare_heads_kernel(float* q_out, const float* proj, long long ld,
+                                                                 const pieh_bias_attn a, const pieh_batch b) {
+  pdl_sync();
+  const long long wi = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
+  const int lane = threadIdx.x & 31, per = a.H + 2 * a.G;
+  if (wi >= (long long)b.T * per) return;
+  const int t = (int)(wi / per), n = (int)(wi - (long long)t * per);
+  const int i = b.tok_seq[t], p = b.tok_pos[t], d = a.d;
+  const float* row = proj + (size_t)t * ld;
+  const size_t slot = (size_t)b.block_table[(size_t)i * b.bt_stride + p / kPage] * kPage + p % kPage;
+  if (n >= a.H + a.G) {
+    const int c0 = (n - a.H - a.G) * a.dv;
+    KT* vp = reinterpret_cast<KT*>(a.v_pages) + slot * a.G * a.dv + c0;
+    const float lam = a.v_mix ? *a.v_mix : 0.f;
+    for (int c = lane; c < a.dv; c += 32) {
+      float v = row[a.v_off + c0 + c];
+      if (a.v_mix) v = (1.f - lam) * v + lam * a.v_keep[(size_t)t * a.G * a.dv + c0 + c];
+      else if (a.v_keep) a.v_keep[(size_t)t * a.G * a.dv + c0 + c] = v;
+      elem<KT>::store(vp + c, v);
+    }
+    return;
+  }
+  const bool is_q = n < a.H;
+  const float* x = is_q ? row + (size_t)n * d : row + a.k_off + (size_t)(n - a.H) * d;
+  const float* nw = is_q ? a.q_norm : a.k_norm;
+  float* qo = q_out + (size_t)t * a.H * d + (size_t)n * d;
+  KT* ko = reinterpret_cast<KT*>(a.k_pages) + (slot * a.G + (is_q ? 0 : n - a.H)) * d;
+  float inv = 1.f;
+  if (nw) {
+    float ss = 0.f;
+    for (int c = lane; c < d; c += 32) ss = fmaf(x[c], x[c], ss);
+    inv = 1.f / sqrtf(warp_sum(ss) / (float)d + a.eps);
+  }
+  if (is_q && a.temp_every > 0.0) inv *= 1.f + a.temp_coef * logf((float)floor((double)(p + 1) / a.temp_every) + 1.f);
+  const int half = a.rot_dims >> 1;
+  const float* cs = a.rot_cs ? a.rot_cs + (size_t)t * half * 2 : nullptr;
+  auto put = [&](int c, float v) { if (is_q) qo[c] = v; else elem<KT>::store(ko + c, v); };
+  for (int e = lane; e < d - half; e += 32) {   // one item per rotated pair, then one per feature that passes through
+    if (e < half) {
+      const int f0 = a.rot_pairs ? 2 * e : e, f1 = a.rot_pairs ? 2 * e + 1 : e + half;
+      const float u = x[f0] * inv * (nw ? nw[f0] : 1.f), v = x[f1] * inv * (nw ? nw[f1] : 1.f);
+      const float co = cs[2 * e], si = cs[2 * e + 1];
+      put(f0, u * co - v * si);
+      put(f1, v * co + u * si);
+    } else {
+      const int f = e + half;
+      put(f, x[f] * inv * (nw ? nw[f] : 1.f));
+    }
+  }
+}
+
 constexpr int kRunWarps = 8;
 
 template <typename T> struct ld8;   // 8 consecutive cache elements as floats
@@ -112,9 +167,11 @@ __global__ void __launch_bounds__(kRunWarps * 32) bias_run_kernel(OT* out, const
   for (int c = threadIdx.x; c < d; c += NTH) qs[c] = q[(size_t)t * a.q_ld + (size_t)h * d + c];
   __syncthreads();
   const int lo = a.window > 0 ? max(0, p - a.window + 1) : 0;
-  // this CTA's slice of the keys lo .. p: whole 32-key blocks, in order of rank
-  const int chunk = ((p - lo + cs) / cs + 31) / 32 * 32;
-  const int my_lo = lo + rank * chunk, my_hi = min(p, my_lo + chunk - 1);
+  // the visible keys in order: the kept first ones that the window has left behind, then lo .. p; number n is position
+  // n < kept ? n : n + gap.  This CTA's slice of the numbers: whole 32-key blocks, in order of rank
+  const int kept = min(a.keep_first, lo), gap = lo - kept, last = p - gap;
+  const int chunk = ((last + cs) / cs + 31) / 32 * 32;
+  const int my_lo = rank * chunk, my_hi = min(last, my_lo + chunk - 1);
   const float slope = a.slopes ? a.slopes[h] : 0.f;
   // sigmoid weights: no maximum, no denominator -- every partial result is a plain sum (m stays 0, so every merge factor is 1)
   const bool sgm = a.sigmoid != 0;
@@ -127,8 +184,8 @@ __global__ void __launch_bounds__(kRunWarps * 32) bias_run_kernel(OT* out, const
 #pragma unroll
   for (int x = 0; x < NV; ++x) acc[x] = 0.f;
   for (int base = my_lo + warp * 32; base <= my_hi; base += NW * 32) {
-    const int j = base + lane;
-    const bool ok = j <= my_hi;
+    const int n_key = base + lane, j = n_key < kept ? n_key : n_key + gap;
+    const bool ok = n_key <= my_hi;
     long long slot = 0;
     float s = -1e30f;
     if (ok) {
@@ -249,7 +306,7 @@ __global__ void __launch_bounds__(kRunWarps * 32) bias_run_kernel(OT* out, const
 
 // ---- prompt portions on the tensor cores ---------------------------------------------------------------------------
 // A CTA of 4 warps owns one 64-row query tile (consecutive positions of ONE sequence) of one query head; key tiles are
-// whole pages (64 keys) from the first page the window reaches to the page of the tile's last row, double-buffered in
+// whole pages (64 keys): those of the kept first keys, then from the first page the window reaches to the tile's last row, double-buffered in
 // XOR-swizzled shared memory by cp.async.  S = Q K^T on mma.sync.m16n8k16 (bf16 in, fp32 out); scale, distance bias,
 // causal and window mask, online softmax in fp32 (exp2 domain) whose running maximum starts at the sink's score 0, P
 // rounded to bf16, O += P V.  The end adds the sink to the denominator, applies the output gate and stores bf16.
@@ -296,15 +353,17 @@ __global__ void __launch_bounds__(128) bias_tile_kernel(__nv_bfloat16* out, cons
   const int kvh = h / (a.H / a.G);
   const int last_key = pos0 + nrows - 1;
   const int first_key = a.window > 0 ? max(0, pos0 - a.window + 1) : 0;
-  const int j_lo = first_key / kPage, j_hi = last_key / kPage;
+  // the pages to walk: those that hold kept first keys and lie below the window, then the window's own
+  const int w_page = first_key / kPage, k_pages = min(w_page, (a.keep_first + kPage - 1) / kPage), skip = w_page - k_pages;
+  const int j_hi = last_key / kPage - skip;   // walked page n is page n < k_pages ? n : n + skip
   const int32_t* table = b.block_table + (size_t)i * b.bt_stride;
   const __nv_bfloat16* kpool = reinterpret_cast<const __nv_bfloat16*>(a.k_pages);
   const __nv_bfloat16* vpool = reinterpret_cast<const __nv_bfloat16*>(a.v_pages);
   const uint32_t sK = (uint32_t)__cvta_generic_to_shared(smem), sV = SHARED ? sK : sK + 2 * KTILE;
 
   auto issue = [&](int j) {
-    const size_t page = (size_t)table[j] * kPage;
-    const uint32_t dk = sK + ((j - j_lo) & 1) * KTILE, dvv = sV + ((j - j_lo) & 1) * VTILE;
+    const size_t page = (size_t)table[j < k_pages ? j : j + skip] * kPage;
+    const uint32_t dk = sK + (j & 1) * KTILE, dvv = sV + (j & 1) * VTILE;
     constexpr int CK = D / 8, CV = DV / 8;
     for (int e = tid; e < 64 * CK; e += 128) {
       const int r = e / CK, c = e - r * CK;
@@ -317,7 +376,7 @@ __global__ void __launch_bounds__(128) bias_tile_kernel(__nv_bfloat16* out, cons
       }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  issue(j_lo);
+  issue(0);
 
   // Q fragments: rows 16 warp + g and + 8 of the tile (rows past the tile's end repeat its last row)
   const int r0 = warp * 16 + g, r1 = r0 + 8;
@@ -349,11 +408,11 @@ __global__ void __launch_bounds__(128) bias_tile_kernel(__nv_bfloat16* out, cons
   const int w0 = a.window > 0 ? p0 - a.window + 1 : 0, w1 = a.window > 0 ? p1 - a.window + 1 : 0;
   const float slope = a.slopes ? a.slopes[h] : 0.f;
 
-  for (int j = j_lo; j <= j_hi; ++j) {
+  for (int j = 0; j <= j_hi; ++j) {
     if (j < j_hi) { issue(j + 1); asm volatile("cp.async.wait_group 1;" ::: "memory"); }
     else asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
-    const uint32_t tk = sK + ((j - j_lo) & 1) * KTILE, tv = SHARED ? tk : sV + ((j - j_lo) & 1) * VTILE;
+    const uint32_t tk = sK + (j & 1) * KTILE, tv = SHARED ? tk : sV + (j & 1) * VTILE;
     float s[NT][4];
 #pragma unroll
     for (int n = 0; n < NT; ++n) { s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f; }
@@ -367,7 +426,7 @@ __global__ void __launch_bounds__(128) bias_tile_kernel(__nv_bfloat16* out, cons
         mma_16816(s[n], qf[kc + 1][0], qf[kc + 1][1], qf[kc + 1][2], qf[kc + 1][3], b2, b3);
       }
     }
-    const int key0 = j * kPage + 2 * t4;
+    const int key0 = (j < k_pages ? j : j + skip) * kPage + 2 * t4;
     float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
     for (int n = 0; n < NT; ++n) {
@@ -376,7 +435,7 @@ __global__ void __launch_bounds__(128) bias_tile_kernel(__nv_bfloat16* out, cons
       for (int e = 0; e < 4; ++e) {
         const int key = k + (e & 1), pr = e < 2 ? p0 : p1, wl = e < 2 ? w0 : w1;
         const float v = s[n][e] * a.scale - slope * (float)(pr - key);
-        s[n][e] = (key <= pr && key >= wl) ? v * kLog2e : -INFINITY;
+        s[n][e] = (key <= pr && (key >= wl || key < a.keep_first)) ? v * kLog2e : -INFINITY;
       }
       mx0 = fmaxf(mx0, fmaxf(s[n][0], s[n][1]));
       mx1 = fmaxf(mx1, fmaxf(s[n][2], s[n][3]));
@@ -442,14 +501,18 @@ __global__ void __launch_bounds__(128) bias_tile_kernel(__nv_bfloat16* out, cons
   const size_t goff = a.g_off + (a.gate_heads ? (size_t)h : (size_t)h * DV);
   const float* g0 = a.g_off >= 0 ? proj + (size_t)(row0 + min(r0, nrows - 1)) * ld + goff : nullptr;
   const float* g1 = a.g_off >= 0 ? proj + (size_t)(row0 + min(r1, nrows - 1)) * ld + goff : nullptr;
-  const int gs = a.gate_heads ? 0 : 1;   // one logit per head, or one per output feature
+  const bool per_head = a.gate_heads != 0;   // one logit per head, or one per output feature
+  if (g0 && per_head) {
+    inv[0] *= 1.f / (1.f + __expf(-g0[0]));
+    inv[1] *= 1.f / (1.f + __expf(-g1[0]));
+  }
 #pragma unroll
   for (int x = 0; x < DT; ++x) {
     const int c = x * 8 + 2 * t4;
     float y0 = o[x][0] * inv[0], y1 = o[x][1] * inv[0], y2 = o[x][2] * inv[1], y3 = o[x][3] * inv[1];
-    if (g0) {
-      y0 *= 1.f / (1.f + __expf(-g0[gs * c])); y1 *= 1.f / (1.f + __expf(-g0[gs * (c + 1)]));
-      y2 *= 1.f / (1.f + __expf(-g1[gs * c])); y3 *= 1.f / (1.f + __expf(-g1[gs * (c + 1)]));
+    if (g0 && !per_head) {
+      y0 *= 1.f / (1.f + __expf(-g0[c])); y1 *= 1.f / (1.f + __expf(-g0[c + 1]));
+      y2 *= 1.f / (1.f + __expf(-g1[c])); y3 *= 1.f / (1.f + __expf(-g1[c + 1]));
     }
     if (r0 < nrows) *reinterpret_cast<uint32_t*>(out + ((size_t)(row0 + r0) * a.H + h) * DV + c) = pack2(y0, y1);
     if (r1 < nrows) *reinterpret_cast<uint32_t*>(out + ((size_t)(row0 + r1) * a.H + h) * DV + c) = pack2(y2, y3);
@@ -487,7 +550,8 @@ static bool bias_attn_ok(const pieh_bias_attn* a) {
   return a && a->H > 0 && a->G > 0 && a->H % a->G == 0 && a->d > 0 && a->dv > 0 && a->dv <= 512 && a->d <= 1024 &&
          a->k_pages && a->v_pages && a->temp_every >= 0.0 && a->window >= 0 && a->k_off >= 0 && a->v_off >= 0 &&
          a->rot_dims >= 0 && a->rot_dims <= a->d && (a->rot_dims & 1) == 0 && (a->rot_dims == 0 || a->rot_cs) &&
-         (!a->v_mix || a->v_keep) && (a->sigmoid == 0 || a->sigmoid == 1) && a->q_ld >= 0 && a->v_ld >= 0;
+         (!a->v_mix || a->v_keep) && (a->sigmoid == 0 || a->sigmoid == 1) && a->q_ld >= 0 && a->v_ld >= 0 && a->keep_first >= 0 &&
+         (a->keep_first == 0 || a->window > 0);
 }
 
 template <typename KT, typename OT, int NV>
@@ -537,6 +601,13 @@ extern "C" int pieh_bias_attn_prepare(float* q_out, const float* proj, long long
   if (!bias_attn_ok(a)) return PIE_EINVAL_SHAPE;
   if (b->T == 0) return PIE_OK;
   count_launch();
+  if (a->head_norm || a->rot_pairs) {
+    if (!a->head_norm && (a->q_norm || a->k_norm)) return PIE_EUNSUPPORTED;   // adjacent pairs come with per-head norms or none
+    const long long warps = (long long)b->T * (a->H + 2 * a->G);
+    PIEH_DISPATCH_DTYPE(a->kv_dtype, KT, launch_k(bias_prepare_heads_kernel<KT>, dim3((unsigned)((warps + 7) / 8)), dim3(256), 0,
+                                                  (cudaStream_t)stream, q_out, proj, ld, *a, *b));
+    return status_of(cudaGetLastError());
+  }
   PIEH_DISPATCH_DTYPE(a->kv_dtype, KT, launch_k(bias_prepare_kernel<KT>, dim3(b->T), dim3(256), 0, (cudaStream_t)stream, q_out, proj, ld, *a, *b));
   return status_of(cudaGetLastError());
 }

@@ -58,12 +58,20 @@ struct LinArgs {
   const float* gate = nullptr;              // SIGMUL: fp32 logits, element z * gate_bs + m * gate_ld + n
   long long gate_ld = 0, gate_bs = 0;
   int nb = 1;
+  int glu_fn = 0;                           // GLU: 0 the gate is g sigmoid(epi_b g), 1 the tanh form of gelu
 };
+
+// z / 2 (1 + tanh(u)) = z sigmoid(2 u) with u = sqrt(2 / pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gelu_f(float z) {
+  const float u = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);
+  return z / (1.f + expf(-2.f * u));
+}
 
 // the gated pair of PIEH_EPI_GLU: g the gate column, u the linear one
 __device__ __forceinline__ float glu_pair(const LinArgs& a, float g, float u) {
   if (a.epi_a > 0.f) { g = fminf(g, a.epi_a); u = fminf(fmaxf(u, -a.epi_a), a.epi_a); }
-  return g / (1.f + expf(-a.epi_b * g)) * (u + a.epi_c);
+  const float act = a.glu_fn ? gelu_f(g) : g / (1.f + expf(-a.epi_b * g));
+  return act * (u + a.epi_c);
 }
 
 template <typename T> struct elem;
@@ -108,12 +116,6 @@ __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log
 // a z^2 + z / 2 above zero, b (e^z - 1 - z) + z / 2 at and below it (continuous, slope 1/2 at zero from both sides)
 __device__ __forceinline__ float xielu_f(float z, float a, float b) {
   return z > 0.f ? fmaf(a * z, z, 0.5f * z) : fmaf(b, expm1f(z) - z, 0.5f * z);
-}
-
-// z / 2 (1 + tanh(u)) = z sigmoid(2 u) with u = sqrt(2 / pi) (z + 0.044715 z^3)
-__device__ __forceinline__ float gelu_f(float z) {
-  const float u = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);
-  return z / (1.f + expf(-2.f * u));
 }
 
 // out dtype dispatch for host launchers

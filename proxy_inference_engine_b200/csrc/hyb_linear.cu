@@ -349,6 +349,19 @@ extern "C" int pieh_linear_glu(void* out, int out_dtype, long long out_ld, const
   return run_linear(a, out_dtype, x_dtype, w_dtype, (cudaStream_t)stream);
 }
 
+extern "C" int pieh_linear_glu_act(void* out, int out_dtype, long long out_ld, const void* x, int x_dtype, long long x_ld,
+                                   const void* w, int w_dtype, int M, int N, int K, int act, float limit, float up_offset,
+                                   void* stream) {
+  if (!out || !x || !w) return PIE_ENULL;
+  if (M < 0 || N <= 0 || K <= 0 || (N & 1) || limit < 0.f) return PIE_EINVAL_SHAPE;
+  if (act != PIEH_EPI_NONE && act != PIEH_EPI_GELU) return PIE_EUNSUPPORTED;
+  if (M == 0) return PIE_OK;
+  LinArgs a{out, out_ld, x, x_ld, w, nullptr, M, N, K, PIEH_EPI_GLU, limit, nullptr, nullptr, 0};
+  a.epi_c = up_offset;
+  a.glu_fn = act == PIEH_EPI_GELU;
+  return run_linear(a, out_dtype, x_dtype, w_dtype, (cudaStream_t)stream);
+}
+
 extern "C" int pieh_moe_linear(void* out, int out_dtype, long long out_ld, const void* x, int x_dtype, long long x_ld,
                                const void* w, int w_dtype, long long w_stride, int P, int N, int K, int gather_rows, int glu,
                                float alpha, float limit, float up_offset, const pieh_moe_plan* p, void* stream) {

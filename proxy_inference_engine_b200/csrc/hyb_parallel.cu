@@ -369,10 +369,11 @@ __global__ void __launch_bounds__(256) latent_rot_kernel(const float* proj, long
     float* q = a.q_rot + (size_t)t * a.q_rot_ld + (size_t)(h < a.H ? h : 0) * a.q_rot_head;
     KT* kd = page + a.kv_rank;
     if (f < half) {
-      const float u = src[f], v = src[f + half], co = cs[2 * f], si = cs[2 * f + 1];
+      const int f0 = a.rot_pairs ? 2 * f : f, f1 = a.rot_pairs ? 2 * f + 1 : f + half;
+      const float u = src[f0], v = src[f1], co = cs[2 * f], si = cs[2 * f + 1];
       const float x = u * co - v * si, y = v * co + u * si;
-      if (h < a.H) { q[f] = x; q[f + half] = y; }
-      else { elem<KT>::store(kd + f, x); elem<KT>::store(kd + f + half, y); }
+      if (h < a.H) { q[f0] = x; q[f1] = y; }
+      else { elem<KT>::store(kd + f0, x); elem<KT>::store(kd + f1, y); }
     } else {
       const int c = a.rot_n + f - half;
       const float x = src[c];

@@ -58,10 +58,11 @@ from dataclasses import dataclass, field
 import torch
 
 from . import _lib
-from ._lib import (DTYPE_BF16, DTYPE_F32, EPI_GELU, EPI_NONE, HybBiasAttn, HybGla, HybLatentRot, HybMixSum, HybMoePlan)
+from ._lib import DTYPE_BF16, DTYPE_F32, EPI_GELU, EPI_NONE, HybGla, HybMixSum, HybMoePlan
 from .babodra import interleave_pairs
 from .cache import HybridCache
 from .golitar import _Linear, _p, _stream
+from .latent import LatentMixin
 from .ragged import BatchDetails
 
 GLA = ("gla", "gla_2")
@@ -131,13 +132,7 @@ class DuduraxArgs:
                 "postln_alpha": self.alpha, "embedding": emb, "layers": self.layers}
 
 
-def rotary_frequencies(rot: dict) -> list:
-    """Angle per position of rotated pair i: base^(-2 i / dims)."""
-    dims = int(rot["dims"])
-    return [float(rot["base"]) ** (-2.0 * i / dims) for i in range(dims // 2)]
-
-
-class DuduraxModel:
+class DuduraxModel(LatentMixin):
     def __init__(self, args: DuduraxArgs, weights: dict, device="cuda", dtype: str = "bfloat16"):
         if dtype not in ("bfloat16", "float32"):
             raise ValueError("dtype must be 'bfloat16' or 'float32'")
@@ -196,40 +191,6 @@ class DuduraxModel:
         if self.pairs is not None:
             self.cache_specs.append({"int_slots": {"last_token": ()}})     # belongs to the embedding, after the layers' entries
 
-    def _latent_weights(self, ly, m, mw, lin, f32):
-        """Fused projection of a latent-attention layer.  Per head the query is taken into the latent space by uk^T: where the
-        latent is no wider than a head's unrotated part, uk^T q is one matrix of no more rows; likewise o uv on the way out."""
-        H, d, dr, dv, r = (int(m[k]) for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank"))
-        if r > 512 or r + dr > 1024:
-            raise ValueError(f"kv_rank {r} + rot_dim {dr} is beyond what the latent attention kernel holds (512 + 512)")
-        W, wdt = self.W, torch.float32 if self.exact else torch.bfloat16
-        ly["dims"] = (H, d, dr, dv, r)
-        ukT = mw("uk").reshape(H, d, r).transpose(1, 2)                       # [H, r, d]
-        qh = mw("q").reshape(H, d + dr, W)
-        ly["ukT"] = ly["uv"] = None
-        if r <= d:
-            q_lat = torch.bmm(ukT.double(), qh[:, :d].double()).float()
-            qw = torch.cat([q_lat, qh[:, d:].float()], 1)                     # [H, r + dr, W]
-        else:
-            qw, ly["ukT"] = qh.float(), ukT.to(device=self.device, dtype=wdt).contiguous()
-        ly["proj"] = lin(torch.cat([qw.reshape(-1, W), mw("dkv").float()], 0))
-        ly["q_rows"] = qw.shape[1]                                            # projection rows per head
-        uv = mw("uv").reshape(H, dv, r)
-        if r <= dv:
-            o = mw("o").reshape(W, H, dv).permute(1, 0, 2)                    # [H, W, dv]
-            ly["out"] = lin(torch.bmm(o.double(), uv.double()).permute(1, 0, 2).reshape(W, H * r).float())
-        else:
-            ly["uv"], ly["out"] = uv.to(device=self.device, dtype=wdt).contiguous(), lin(mw("o"))
-        ly["kv_norm"], ly["scale"] = f32(mw("dkv.norm")), float(m["scale"])
-        ly["window"] = int((m.get("mask") or {}).get("size") or 0)
-        rot = m.get("rot") or None
-        ly["rot"] = None
-        if rot and int(rot["dims"]) > 0:
-            key = (int(rot["dims"]), float(rot["base"]))
-            if key not in self.rot_tables:
-                self.rot_tables[key] = torch.tensor(rotary_frequencies(rot), dtype=torch.float64).to(self.device)
-            ly["rot"] = key
-
     # ------------------------------------------------------------------------------------------------
     def make_cache(self, max_tokens: int, max_seqs: int = 4) -> HybridCache:
         return HybridCache(self.cache_specs, max_tokens, max_seqs, self.device, self.act_torch, lib=self.L)
@@ -244,28 +205,11 @@ class DuduraxModel:
                                                  lin.w_dtype, _p(lin.bias), M, lin.N, lin.K, act, 0.0, 0.0, _stream()), "linear")
         return out
 
-    def _heads(self, out, out_dtype, out_head, x, w, M, nb, N, K):
-        """nb per-head products in one launch: x [M, nb * K] (head-major columns), w [nb, N, K] -> head z at out + z * out_head."""
-        wd = DTYPE_F32 if self.exact else DTYPE_BF16
-        _lib.check_hybrid(self.L.pieh_linear_batched(_p(out), out_dtype, out.stride(0), out_head, _p(x), self.act, x.stride(0), K,
-                                                     _p(w), wd, N * K, nb, M, N, K, EPI_NONE, None, 0, 0, _stream()),
-                          "linear_batched")
-        return out
-
     def _sum_norm(self, x, h, y, mix, w, T):
         """x <- rms(alpha x + y | mixture) w, h <- x in the act dtype (exact mode: h is x)."""
         _lib.check_hybrid(self.L.pieh_sum_norm(_p(x), None if self.exact else _p(h), self.act, _p(y), C.byref(mix) if mix else None,
                                                _p(w), float(self.args.alpha), float(self.args.norm_eps), T, self.W, _stream()),
                           "sum_norm")
-
-    def _rot(self, key, batch, T, cache):
-        """(cos, sin) table of this step for one (dims, base), formed once and shared by the layers that use it."""
-        if key not in cache:
-            cs = self._empty((T, key[0] // 2, 2))
-            _lib.check_hybrid(self.L.pieh_rot_table(_p(cs), _p(batch.positions), _p(self.rot_tables[key]), T, key[0] // 2,
-                                                    _stream()), "rot_table")
-            cache[key] = cs
-        return cache[key]
 
     def _segment_tiles(self, desc, H, dv):
         """64-row tiles per segment of the scan: enough segments that all heads' column blocks fill the GPU about four times."""
@@ -295,32 +239,6 @@ class DuduraxModel:
                                           _stream()), "gla_scan")
         _lib.check_hybrid(L.pieh_gated_group_norm(_p(mixed), self.act, _p(o), o.stride(0), C.c_void_p(proj.data_ptr() + 4 * g_off),
                                                   ld, _p(ly["all_norm"]), H, dv, eps, 2, 0, T, _stream()), "gated_group_norm")
-        return self._linear(ly["out"], mixed, T)
-
-    def _latent(self, ly, st, h, batch, desc, T, rot_cache):
-        L, eps = self.L, float(self.args.norm_eps)
-        H, d, dr, dv, r = ly["dims"]
-        bref, D = C.byref(desc), r + dr
-        proj = self._linear(ly["proj"], h, T)                  # per head [query | positional part], then [latent | shared key part]
-        ld, kv_off = proj.stride(0), H * ly["q_rows"]
-        rot_n = ly["rot"][0] if ly["rot"] else 0
-        cs = self._rot(ly["rot"], batch, T, rot_cache) if ly["rot"] else None
-        if ly["ukT"] is None:                                  # queries are in the latent space already: rotate them in place
-            q, q_ld, plain, rot_at = proj, ld, None, r
-        else:
-            q, plain, rot_at = self._empty((T, H * D)), self._empty((T, H * d), self.act_torch), d
-            q_ld = q.stride(0)
-        lr = HybLatentRot(H, r, dr, rot_n, 0, ly["q_rows"], rot_at, kv_off, _p(ly["kv_norm"]), eps, _p(cs),
-                          C.c_void_p(q.data_ptr() + 4 * r), q_ld, D, _p(plain), self.act, _p(st["c"]), self.act)
-        _lib.check_hybrid(L.pieh_latent_rot_prepare(_p(proj), ld, C.byref(lr), bref, _stream()), "latent_rot_prepare")
-        if plain is not None:
-            self._heads(q, DTYPE_F32, D, plain, ly["ukT"], T, H, r, d)
-        at = HybBiasAttn(H=H, G=1, d=D, dv=r, g_off=-1, eps=eps, scale=ly["scale"], window=ly["window"], k_pages=_p(st["c"]),
-                         v_pages=_p(st["c"]), kv_dtype=self.act, q_ld=q_ld, v_ld=D)
-        mixed = self._empty((T, H * r), self.act_torch)
-        _lib.check_hybrid(L.pieh_bias_attn_run(_p(mixed), self.act, _p(q), None, 0, C.byref(at), bref, _stream()), "attn_run")
-        if ly["uv"] is not None:
-            mixed = self._heads(self._empty((T, H * dv), self.act_torch), self.act, dv, mixed, ly["uv"], T, H, dv, r)
         return self._linear(ly["out"], mixed, T)
 
     def _moe(self, ml, h, T):

@@ -1,7 +1,7 @@
 """Continuous-batching engine for models that step over ``ragged.BatchDetails`` with a ``cache.HybridCache``
 (``golitar.GolitarModel``, ``babodra.BabodraModel``, ``maginex.MaginexModel``, ``zelinex.ZelinexModel``,
-``dudurax.DuduraxModel``): the generate loop of PIE (PIE/engine/inference_engine.py:228-297) lifted from one sequence to a
-changing set of them.
+``dudurax.DuduraxModel``, ``vokusun.VokusunModel``): the generate loop of PIE (PIE/engine/inference_engine.py:228-297)
+lifted from one sequence to a changing set of them.
 
     eng = HybridEngine(model, max_tokens=4096, max_seqs=4)
     outs = eng.generate([prompt_a, prompt_b, ...], max_new_tokens=32)           # greedy; sampler=make_sampler(...)
