@@ -17,11 +17,13 @@
 //                       shares one pair: each CTA takes a contiguous slice of the keys and the first CTA of the cluster
 //                       reads the others' partial softmax out of their shared memory (distributed shared memory), so a
 //                       long context is spread over the whole GPU without a workspace or a second launch
+// latent_decode_kernel  (hyb_latent_decode.cu) single tokens over a pool shared by all heads, bf16: the heads are a tile's rows
 // bias_tile_kernel      prompt portions over bf16 pages: 64-row query tiles on mma.sync (below)
 // A step's keys are appended before its queries run, so a prompt portion sees itself through the same pages as its past.
 #include <cooperative_groups.h>
 
 #include "hyb_common.cuh"
+#include "hyb_mma.cuh"
 
 namespace pieh {
 
@@ -310,26 +312,6 @@ __global__ void __launch_bounds__(kRunWarps * 32) bias_run_kernel(OT* out, const
 // XOR-swizzled shared memory by cp.async.  S = Q K^T on mma.sync.m16n8k16 (bf16 in, fp32 out); scale, distance bias,
 // causal and window mask, online softmax in fp32 (exp2 domain) whose running maximum starts at the sink's score 0, P
 // rounded to bf16, O += P V.  The end adds the sink to the denominator, applies the output gate and stores bf16.
-__device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void ldsm_x4_trans(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void mma_16816(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
-                                          uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t pack2(float lo, float hi) {
-  const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-  return *reinterpret_cast<const uint32_t*>(&v);
-}
-__device__ __forceinline__ void cp16(uint32_t dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
-}
 template <int ROWB>   // bytes of a tile row (>= 128); 16-byte chunk c of row r sits at chunk c ^ (r & 7)
 __device__ __forceinline__ uint32_t tile_off(int r, int c) { return (uint32_t)(r * ROWB + ((c ^ (r & 7)) << 4)); }
 
@@ -407,6 +389,8 @@ __global__ void __launch_bounds__(128) bias_tile_kernel(__nv_bfloat16* out, cons
   const int p0 = pos0 + min(r0, nrows - 1), p1 = pos0 + min(r1, nrows - 1);   // positions of this thread's two rows
   const int w0 = a.window > 0 ? p0 - a.window + 1 : 0, w1 = a.window > 0 ? p1 - a.window + 1 : 0;
   const float slope = a.slopes ? a.slopes[h] : 0.f;
+  const float scale2 = a.scale * kLog2e, slope2 = slope * kLog2e;            // scores in the exp2 domain
+  const int w_last = a.window > 0 ? last_key - a.window + 1 : 0;             // where the last row's window begins
 
   for (int j = 0; j <= j_hi; ++j) {
     if (j < j_hi) { issue(j + 1); asm volatile("cp.async.wait_group 1;" ::: "memory"); }
@@ -426,19 +410,29 @@ __global__ void __launch_bounds__(128) bias_tile_kernel(__nv_bfloat16* out, cons
         mma_16816(s[n], qf[kc + 1][0], qf[kc + 1][1], qf[kc + 1][2], qf[kc + 1][3], b2, b3);
       }
     }
-    const int key0 = (j < k_pages ? j : j + skip) * kPage + 2 * t4;
+    const int page0 = (j < k_pages ? j : j + skip) * kPage, key0 = page0 + 2 * t4;
     float mx0 = -INFINITY, mx1 = -INFINITY;
+    if (slope == 0.f && page0 + kPage - 1 <= pos0 && (page0 >= w_last || page0 + kPage <= a.keep_first)) {
 #pragma unroll
-    for (int n = 0; n < NT; ++n) {
-      const int k = key0 + n * 8;
+      for (int n = 0; n < NT; ++n) {   // every row of the tile sees every key of the page
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int key = k + (e & 1), pr = e < 2 ? p0 : p1, wl = e < 2 ? w0 : w1;
-        const float v = s[n][e] * a.scale - slope * (float)(pr - key);
-        s[n][e] = (key <= pr && (key >= wl || key < a.keep_first)) ? v * kLog2e : -INFINITY;
+        for (int e = 0; e < 4; ++e) s[n][e] *= scale2;
+        mx0 = fmaxf(mx0, fmaxf(s[n][0], s[n][1]));
+        mx1 = fmaxf(mx1, fmaxf(s[n][2], s[n][3]));
       }
-      mx0 = fmaxf(mx0, fmaxf(s[n][0], s[n][1]));
-      mx1 = fmaxf(mx1, fmaxf(s[n][2], s[n][3]));
+    } else {
+#pragma unroll
+      for (int n = 0; n < NT; ++n) {
+        const int k = key0 + n * 8;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int key = k + (e & 1), pr = e < 2 ? p0 : p1, wl = e < 2 ? w0 : w1;
+          const float v = fmaf(s[n][e], scale2, -slope2 * (float)(pr - key));
+          s[n][e] = (key <= pr && (key >= wl || key < a.keep_first)) ? v : -INFINITY;
+        }
+        mx0 = fmaxf(mx0, fmaxf(s[n][0], s[n][1]));
+        mx1 = fmaxf(mx1, fmaxf(s[n][2], s[n][3]));
+      }
     }
     uint32_t pf[NT][2];
     if (sgm) {
@@ -546,6 +540,11 @@ static bool tile_ok(const pieh_bias_attn& a, const pieh_batch& b, int out_dtype)
          b.n_tiles > 0 && b.tile_seq && b.tile_row && a.H <= 65535 && (long long)b.T >= 16LL * b.n_seq;
 }
 
+// hyb_latent_decode.cu: the heads of one token as the rows of a tensor-core tile
+bool latent_decode_ok(const pieh_bias_attn& a, const pieh_batch& b);
+cudaError_t launch_latent_decode(__nv_bfloat16* out, const float* q, const float* proj, long long ld, const pieh_bias_attn& a,
+                                 const pieh_batch& b, cudaStream_t st);
+
 static bool bias_attn_ok(const pieh_bias_attn* a) {
   return a && a->H > 0 && a->G > 0 && a->H % a->G == 0 && a->d > 0 && a->dv > 0 && a->dv <= 512 && a->d <= 1024 &&
          a->k_pages && a->v_pages && a->temp_every >= 0.0 && a->window >= 0 && a->k_off >= 0 && a->v_off >= 0 &&
@@ -633,6 +632,9 @@ extern "C" int pieh_bias_attn_run(void* out, int out_dtype, const float* q, cons
 #undef PIEH_TILE
     return status_of(e);
   }
+  static const bool no_latent = [] { const char* v = getenv("PIE_HYBRID_NO_LATENT_DECODE"); return v && v[0] == '1'; }();
+  if (!no_latent && a->kv_dtype == PIE_DTYPE_BF16 && out_dtype == PIE_DTYPE_BF16 && tile_shared(*a) && latent_decode_ok(*a, *b))
+    return status_of(launch_latent_decode((bf*)out, q, proj, ld, *a, *b, st));
   if (a->kv_dtype == PIE_DTYPE_BF16)
     e = out_dtype == PIE_DTYPE_BF16 ? launch_run<bf, bf>((bf*)out, q, proj, ld, *a, *b, st)
                                     : launch_run<bf, float>((float*)out, q, proj, ld, *a, *b, st);

@@ -1,10 +1,13 @@
-"""Throughput of the Golitar, Babodra, Maginex, Zelinex and Dudurax families at layer sizes of real models (random weights), with
-every operator of the step timed in place and set against its roofline.  Golitar is shown beside the quantized Llama path
+"""Throughput of the Golitar, Babodra, Maginex, Zelinex, Dudurax and Vokusun families at layer sizes of real models (random
+weights), with every operator of the step timed in place and set against its roofline.  Golitar is shown beside the quantized Llama path
 at equal width / feed-forward / depth; Babodra beside Golitar, Maginex beside Babodra, and Zelinex beside Golitar (the other
 family built on a matrix-state recurrence and windowed attention), Dudurax beside Maginex (latent attention, recurrence,
-experts in every layer) and Zelinex (matrix-state scans), at equal width / depth / active feed-forward size.
+experts in every layer) and Zelinex (matrix-state scans), at equal width / depth / active feed-forward size; Vokusun beside
+Dudurax (latent attention with a rotated part), Zelinex (looped sandwich blocks, windowed grouped-head attention), Maginex
+(latent attention over all earlier tokens) and Golitar (dense feed-forwards).
 
-``run(size, ...)`` is what ``bench.py --family golitar|babodra|maginex|zelinex|dudurax`` prints.  Method: one prompt of ``prompt`` tokens goes through
+``run(size, ...)`` is what ``bench.py --family golitar|babodra|maginex|zelinex|dudurax|vokusun`` prints.  Method: one prompt of
+``prompt`` tokens goes through
 ``HybridEngine.forward`` in portions of ``portion`` rows (prefill tok/s, CUDA events around all portions), then ``batch``
 sequences decode ``steps`` tokens each (decode tok/s).  The per-operator table wraps every library call of one prefill
 portion and one decode step in a CUDA event pair; bytes and flops are the algorithmic ones of the call's shapes, the
@@ -31,6 +34,8 @@ SIZES = {
                dud=dict(pattern="ggahggahggahggah", gla=(8, 128, 256), gla_2=(4, 256, 512), tau=16.0, heads=16, dim=128,
                         rot_dim=64, vdim=128, kv_rank=128, window=1024, experts=16, identity=4, groups=(5, 3), top=4,
                         expert_ff=2048),
+               vok=dict(pattern="laallaallaal", loop=(0, 4, 2), heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=128, a_heads=16,
+                        a_kv=4, a_dim=128, a_rot=64, window=1024, keep=4),
                llama=dict(hidden_size=2048, intermediate_size=8192, num_attention_heads=32,
                                                        num_key_value_heads=8, head_dim=64, vocab_size=32000)),
     "8b": dict(width=4096, ff=14336, vocab=32000, pattern="dddadddA", dH=32, dG=16, dk=128, dv=128, aH=32, aG=8, ad=64,
@@ -44,6 +49,8 @@ SIZES = {
                dud=dict(pattern="ggahggah", gla=(16, 128, 256), gla_2=(8, 256, 512), tau=16.0, heads=32, dim=128,
                         rot_dim=64, vdim=128, kv_rank=128, window=2048, experts=16, identity=4, groups=(5, 3), top=4,
                         expert_ff=3584),
+               vok=dict(pattern="lalala", loop=(0, 2, 2), heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=128, a_heads=32,
+                        a_kv=8, a_dim=128, a_rot=64, window=2048, keep=4),
                llama=dict(hidden_size=4096, intermediate_size=14336, num_attention_heads=32,
                                                 num_key_value_heads=8, head_dim=128, vocab_size=32000)),
 }
@@ -144,6 +151,23 @@ def dudurax_config(size: str) -> dict:
             "embedding": {"scale": 4.0, "bigram": {"buckets": 32749, "mul_prev": 1009, "mul_cur": 37}}, "layers": layers}
 
 
+def vokusun_config(size: str) -> dict:
+    """Same width and the same number of layer RUNS as the others (part of the stack is looped twice); latent attention over all
+    earlier tokens and windowed attention with kept first tokens, every layer with golitar_config's dense feed-forward size."""
+    s = SIZES[size]
+    v = s["vok"]
+    mixers = {"l": ("latent_attention", {"heads": v["heads"], "dim": v["dim"], "rot_dim": v["rot_dim"], "vdim": v["vdim"],
+                                         "kv_rank": v["kv_rank"], "scale": (v["dim"] + v["rot_dim"]) ** -0.5,
+                                         "rot": {"base": 1e5, "dims": v["rot_dim"]}}),
+              "a": ("attention", {"heads": v["a_heads"], "kv_heads": v["a_kv"], "dim": v["a_dim"], "vdim": v["a_dim"],
+                                  "scale": v["a_dim"] ** -0.5, "mask": {"size": v["window"], "keep_first": v["keep"]},
+                                  "rot": {"base": 1e6, "dims": v["a_rot"], "scaling": {"factor": 4.0}}})}
+    layers = [{"type": mixers[ch][0], "mixer": dict(mixers[ch][1]), "mlp": {"kind": "dense", "ff": s["ff"]}} for ch in v["pattern"]]
+    a, b, t = v["loop"]
+    return {"architecture": "Vokusun", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5},
+            "loop": {"start": a, "stop": b, "times": t}, "layers": layers}
+
+
 def _peaks(root):
     try:
         with open(os.path.join(root, "MEASURED_PEAKS.json")) as f:
@@ -186,7 +210,7 @@ def _cost(name, a, model, batch_info):
         wb = 4 if a[7] == 1 else 2
         extra = 2 * model.S * M * N * 4 if epi == 3 else M * N * ob
         return N * K * wb + M * K * act + extra, 2.0 * M * N * K, f"linear M={M}"
-    if name == "pieh_linear_glu":
+    if name in ("pieh_linear_glu", "pieh_linear_glu_act"):
         M, N, K = a[8], a[9], a[10]
         ob = 4 if a[1] == 1 else 2
         wb = 4 if a[7] == 1 else 2
@@ -214,6 +238,11 @@ def _cost(name, a, model, batch_info):
         adds = (1 if a[5] is not None else 0)
         return (Tn * W * (4 * (parts + adds + 2) + (act if a[7] is not None else 0)), 0.0,
                 "sandwich_add" + ("(mixture)" if mix is not None else ""))
+    if name == "pieh_layernorm_add":
+        n, W = a[14], a[15]
+        rows = (a[1] is not None) + (0 if a[1] is not None and a[3] is None else 1) + (a[5] is not None)      # read
+        rows += 1 if a[12] is None and (a[1] is not None or a[5] is not None or a[7] is not None) else 0         # written
+        return n * W * (4 * rows + (act if a[8] is not None else 0)), 0.0, "layernorm_add"
     if name == "pieh_gated_group_norm":
         return a[12] * a[7] * a[8] * (8 + act), 0.0, "gated_group_norm"
     if name == "pieh_gdelta_prepare":
@@ -278,9 +307,9 @@ def _cost(name, a, model, batch_info):
         own = T // max(n_seq, 1)
         keys = ctx + own
         per_q = ctx + (own + 1) / 2 if T > n_seq else keys
-        if at.window:       # a query sees at most `window` keys; the step reads the pages its first row's window reaches
-            per_q = min(per_q, at.window)
-            keys = min(keys, at.window + own)
+        if at.window:       # a query sees at most `window` keys (+ kept first ones); the step reads what its first row's window reaches
+            per_q = min(per_q, at.window + at.keep_first)
+            keys = min(keys, at.window + at.keep_first + own)
         shared_kv = 1 if at.k_pages == at.v_pages else 2      # latent attention: keys and values are one pool
         kvb = n_seq * keys * G * (d if shared_kv == 1 else d + dv) * act
         return (kvb + T * H * (d * 4 + dv * (act + 4)), 2.0 * T * H * per_q * (d + dv),
@@ -332,7 +361,16 @@ def run(size="1b", prompt=4096, portion=4096, batch=4, steps=32, warmup=3, root=
 
     hbm, tfl, src = _peaks(root)
     t0 = time.time()
-    if family == "dudurax":
+    if family == "vokusun":
+        from .vokusun import VokusunArgs, VokusunModel, random_weights
+        cfg = vokusun_config(size)
+        args = VokusunArgs.from_dict(cfg)
+        weights = random_weights(args, seed=0, device="cuda")
+        n_params = sum(v.numel() for v in weights.values())
+        model = VokusunModel(args, weights, "cuda", "bfloat16")
+        del weights
+        pattern = "".join(SIZES[size]["vok"]["pattern"][i] for i, _ in args.runs())
+    elif family == "dudurax":
         from .dudurax import DuduraxArgs, DuduraxModel, random_weights
         cfg = dudurax_config(size)
         args = DuduraxArgs.from_dict(cfg)
@@ -429,7 +467,11 @@ def run(size="1b", prompt=4096, portion=4096, batch=4, steps=32, warmup=3, root=
            "pipeline_error": int(timed._lib.pieh_pipeline_error()), "setup_s": round(time.time() - t0, 1)}
     del eng, model
     torch.cuda.empty_cache()
-    if family == "dudurax":
+    if family == "vokusun":
+        if with_llama:      # the families whose operators are closest, at the same width and number of layer runs
+            for other in ("dudurax", "zelinex", "maginex", "golitar"):
+                out[f"{other}_equal_size"] = run(size, prompt, portion, batch, steps, warmup, root, with_llama=False, family=other)
+    elif family == "dudurax":
         if with_llama:      # the closest models of the framework at the same sizes: latent attention, recurrence and experts in
             for other in ("maginex", "zelinex"):                 # every layer; matrix-state scans
                 out[f"{other}_equal_size"] = run(size, prompt, portion, batch, steps, warmup, root, with_llama=False, family=other)
